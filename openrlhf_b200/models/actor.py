@@ -12,6 +12,7 @@ import torch.nn as nn
 
 from .config import ModelConfig
 from .packing import PackedBatch, pack_padded, unpack_to_padded
+from .registry import require_trainable
 from .transformer import TransformerLM
 
 
@@ -42,6 +43,7 @@ class Actor(nn.Module):
 
             self.model = load_pretrained(pretrain_or_model, device=device, shard_world=shard_world, seed=seed)
         self.cfg: ModelConfig = self.model.cfg
+        require_trainable(self.cfg)
         self.lora = None
         if lora_rank and lora_rank > 0:
             from .lora import LoraAdapters

@@ -2,10 +2,11 @@
 definition needs, with converters from and to ``config.json`` and presets for the benchmark architectures."""
 from __future__ import annotations
 
-import dataclasses
 import json
 import os
 from dataclasses import dataclass, field
+
+from .hybrid_config import sigisun_preset
 
 
 @dataclass
@@ -167,10 +168,10 @@ class ModelConfig:
 
     @classmethod
     def from_pretrained(cls, path: str) -> "ModelConfig":
-        if path in PRESETS:
-            return dataclasses.replace(PRESETS[path])
-        with open(os.path.join(path, "config.json")) as f:
-            return cls.from_hf_dict(json.load(f))
+        """Configuration of a preset or a checkpoint folder (``models/registry.py`` picks the reader)."""
+        from .registry import read_config
+
+        return read_config(path)
 
     def save_pretrained(self, path: str, extra: dict | None = None) -> None:
         os.makedirs(path, exist_ok=True)
@@ -216,3 +217,10 @@ PRESETS: dict[str, ModelConfig] = {
     "tiny-qwen3-moe": ModelConfig("qwen3_moe", 1024, 128, 256, 2, 2, 1, head_dim=128, rope_theta=1e6, num_experts=8,
                                   num_experts_per_tok=2, moe_intermediate_size=64, norm_topk_prob=True, qk_norm=True),
 }
+
+# served designs with their own layer lists (models/hybrid_config.py)
+PRESETS.update({
+    "tiny-sigisun": sigisun_preset(192, 6, 6, 32, 48, 2, 6, 2, 48, 40, 3, 224, 512),
+    "sigisun-1b": sigisun_preset(2048, 24, 64, 64, 128, 1, 16, 4, 128, 1024, 4, 4096, 65536),
+    "sigisun-8b": sigisun_preset(4096, 36, 128, 64, 128, 8, 32, 8, 128, 2048, 4, 11008, 128256),
+})

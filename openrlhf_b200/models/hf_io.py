@@ -17,6 +17,8 @@ from typing import Iterator
 import torch
 
 from .config import PRESETS, ModelConfig
+from .flat import FlatModel
+from .registry import build_model, read_config
 from .transformer import TransformerLM
 
 MAX_SHARD_BYTES = 5 * 1024 ** 3
@@ -25,9 +27,11 @@ MAX_SHARD_BYTES = 5 * 1024 ** 3
 def hf_names_for(cfg: ModelConfig, name: str) -> list[tuple[str, tuple | None]]:
     """Internal parameter name -> [(hf_name, row slice or expert selector)].
 
-    A selector is None (whole tensor), ("rows", a, b) for a row range of a fused matrix / bias, or
-    ("expert", e, a, b) for rows [a, b) of expert e of a fused 3-D tensor.
+    A selector is None (whole tensor), ("rows", a, b) for a row range of a fused matrix / bias, ("block", r0, r1, c0,
+    c1) for rows and columns of one, or ("expert", e, a, b) for rows [a, b) of expert e of a fused 3-D tensor.
     """
+    if hasattr(cfg, "checkpoint_names"):      # a design with a checkpoint layout of its own
+        return cfg.checkpoint_names(name)
     if name.startswith("visual."):
         # vision tower (Qwen2-VL): same names under "model."; the patch embedding is stored as a Conv3d kernel
         if name == "visual.patch_embed.weight":
@@ -96,6 +100,8 @@ def _select(t: torch.Tensor, sel):
         return t
     if sel[0] == "rows":
         return t[sel[1]:sel[2]]
+    if sel[0] == "block":
+        return t[sel[1]:sel[2], sel[3]:sel[4]]
     if sel[0] == "view":
         return t.reshape(sel[1])
     return t[sel[1], sel[2]:sel[3]]
@@ -221,20 +227,18 @@ def load_weights(model: TransformerLM, path: str, strict: bool = True) -> list[s
 
 def load_pretrained(path_or_preset: str, device="cuda", with_lm_head: bool = True, with_value_head: bool = False,
                     shard_world: int = 1, seed: int = 0, init_value_head: bool = False,
-                    value_head_prefix: str | None = None) -> TransformerLM:
+                    value_head_prefix: str | None = None, dtype: torch.dtype | None = None) -> FlatModel:
     """Build a model from an HF checkpoint directory, or random-init it from an architecture preset name
     (``qwen2.5-1.5b``, ``llama3-8b``, ...; presets exist because the benchmark machines have no network)."""
-    if path_or_preset in PRESETS:
-        cfg = ModelConfig.from_pretrained(path_or_preset)
-        if value_head_prefix:
-            cfg.value_head_prefix = value_head_prefix
-        return TransformerLM(cfg, device=device, with_lm_head=with_lm_head, with_value_head=with_value_head,
-                             seed=seed, shard_world=shard_world)
-    cfg = ModelConfig.from_pretrained(path_or_preset)
+    cfg = read_config(path_or_preset)
     if value_head_prefix:
         cfg.value_head_prefix = value_head_prefix
-    model = TransformerLM(cfg, device=device, with_lm_head=with_lm_head, with_value_head=with_value_head, seed=None,
-                          shard_world=shard_world)
+    kw = {} if dtype is None else {"dtype": dtype}
+    preset = path_or_preset in PRESETS
+    model = build_model(cfg, device=device, with_lm_head=with_lm_head, with_value_head=with_value_head,
+                        seed=seed if preset else None, shard_world=shard_world, **kw)
+    if preset:
+        return model
     if with_value_head:
         g = torch.Generator(device="cpu").manual_seed(seed)
         vh = model.p("value_head.weight")

@@ -9,7 +9,6 @@ parameters are views into one flat bf16 buffer (the unit of ZeRO sharding, weigh
 from __future__ import annotations
 
 import math
-from dataclasses import dataclass
 
 import torch
 import torch.nn as nn
@@ -17,30 +16,12 @@ import torch.utils.checkpoint
 
 from ..ops import functional as F
 from .config import ModelConfig
-
-ALIGN = 128  # every parameter starts on a 256-byte boundary of the flat buffer (TMA needs 16 B; shards like 256 B)
-
-
-@dataclass
-class ParamSpec:
-    name: str
-    shape: tuple
-    offset: int
-    numel: int
-    decay: bool       # subject to weight decay (matrices) or exempt (norms, biases)
-    init: str         # normal | ones | zeros
+from .flat import ALIGN, FlatModel, ParamSpec, SpecList  # noqa: F401  (re-exported: the training engines import them here)
 
 
 def build_param_specs(cfg: ModelConfig, with_lm_head: bool = True, with_value_head: bool = False) -> list[ParamSpec]:
-    specs: list[ParamSpec] = []
-    off = 0
-
-    def add(name, shape, decay=True, init="normal"):
-        nonlocal off
-        n = math.prod(shape)
-        specs.append(ParamSpec(name, tuple(shape), off, n, decay, init))
-        off += (n + ALIGN - 1) // ALIGN * ALIGN
-
+    layout = SpecList()
+    add = layout.add
     H = cfg.hidden_size
     add("embed.weight", (cfg.vocab_size, H))
     for i in range(cfg.num_hidden_layers):
@@ -72,10 +53,10 @@ def build_param_specs(cfg: ModelConfig, with_lm_head: bool = True, with_value_he
 
         for name, shape, decay, init in vision_param_shapes(cfg.vision_config()):
             add(name, shape, decay, init)
-    return specs
+    return layout.specs
 
 
-class TransformerLM(nn.Module):
+class TransformerLM(FlatModel):
     """Decoder stack over a packed token stream. ``forward`` returns the final-norm hidden states [T, H]."""
 
     def __init__(self, cfg: ModelConfig, device="cpu", dtype=torch.bfloat16, with_lm_head=True, with_value_head=False,
@@ -83,22 +64,8 @@ class TransformerLM(nn.Module):
                  shard_world: int = 1):
         super().__init__()
         self.cfg = cfg
-        self.specs = build_param_specs(cfg, with_lm_head, with_value_head)
         self.with_lm_head, self.with_value_head = with_lm_head, with_value_head
-        total = self.specs[-1].offset + (self.specs[-1].numel + ALIGN - 1) // ALIGN * ALIGN
-        if flat is None:
-            # room for the padding that makes the flat index space divisible into `shard_world` aligned shards
-            per = ((total + shard_world - 1) // shard_world + 255) // 256 * 256
-            flat = torch.zeros(per * shard_world, dtype=dtype, device=device)
-        assert flat.numel() >= total
-        self.flat = flat                      # not a Parameter: parameters are views into it
-        self.total_numel = total
-        self._params: dict[str, nn.Parameter] = {}
-        for s in self.specs:
-            view = flat[s.offset:s.offset + s.numel].view(s.shape)
-            p = nn.Parameter(view, requires_grad=True)
-            self._params[s.name] = p
-            self.register_parameter(s.name.replace(".", "__"), p)
+        self.init_flat(build_param_specs(cfg, with_lm_head, with_value_head), device, dtype, flat, shard_world)
         self.gradient_checkpointing = False
         self.tp_group = None   # set on a tensor-parallel shard of the model (rollout/tp_engine.py)
         self.tp_train = None   # parallel.tp_train.TPTrain: this model is one rank's shard of a TP-trained model
@@ -110,31 +77,13 @@ class TransformerLM(nn.Module):
             self.reset_parameters(init_std, seed)
 
     # ------------------------------------------------------------------ parameters
-    def p(self, name: str) -> nn.Parameter:
-        return self._params[name]
-
-    def named_specs(self):
-        return [(s, self._params[s.name]) for s in self.specs]
-
-    @torch.no_grad()
-    def reset_parameters(self, std: float = 0.02, seed: int = 0):
-        g = torch.Generator(device=self.flat.device).manual_seed(seed)
-        for s, p in self.named_specs():
-            if s.init == "ones":
-                p.fill_(1.0)
-            elif s.init == "zeros":
-                p.zero_()
-            elif s.name == "value_head.weight":
-                # N(0, 1/(hidden+1)) as in openrlhf/models/model.py:164-172
-                p.copy_(torch.randn(s.shape, generator=g, device=p.device, dtype=torch.float32)
-                        * (1.0 / math.sqrt(self.cfg.hidden_size + 1)))
-            else:
-                # chunked to bound the fp32 temporary for large embeddings
-                flat = p.view(-1)
-                step = 1 << 26
-                for a in range(0, flat.numel(), step):
-                    b = min(flat.numel(), a + step)
-                    flat[a:b].copy_(torch.randn(b - a, generator=g, device=p.device, dtype=torch.float32) * std)
+    def init_special(self, s: ParamSpec, p: nn.Parameter, g: torch.Generator) -> bool:
+        if s.name != "value_head.weight":
+            return False
+        # N(0, 1/(hidden+1)) as in openrlhf/models/model.py:164-172
+        p.copy_(torch.randn(s.shape, generator=g, device=p.device, dtype=torch.float32)
+                * (1.0 / math.sqrt(self.cfg.hidden_size + 1)))
+        return True
 
     def lm_head_weight(self) -> torch.Tensor:
         return self.p("embed.weight") if self.cfg.tie_word_embeddings else self.p("lm_head.weight")

@@ -34,16 +34,36 @@ class KernelError(RuntimeError):
     """A kernel reported a non-zero status word (for instance a bounded wait that ran out)."""
 
 
+_component: str | None = None
+
+
+def prefer_component(name: str) -> None:
+    """Before the first kernel: if the full library is not built, use (and if need be build) this component of it
+    (``csrc.build.COMPONENTS``) instead. A symbol outside the component raises AttributeError."""
+    global _component
+    if _lib is None and not os.path.exists(LIB_PATH):
+        _component = name
+
+
+def lib_path() -> str:
+    """The library this process uses, or would use once built."""
+    if _component is None:
+        return LIB_PATH
+    from openrlhf_b200.csrc.build import component_path
+
+    return component_path(_component)
+
+
 def lib() -> ctypes.CDLL:
     global _lib
     if _lib is None:
         with _lock:
             if _lib is None:
-                if not os.path.exists(LIB_PATH):
+                if not os.path.exists(lib_path()):
                     from openrlhf_b200.csrc.build import build
 
-                    build()
-                _lib = ctypes.CDLL(LIB_PATH)
+                    build(component=_component)
+                _lib = ctypes.CDLL(lib_path())
     return _lib
 
 

@@ -91,3 +91,84 @@ def paged_decode_attention(q, k_cache, v_cache, block_table, seq_lens, scale, pa
         att = torch.einsum("hd,hld->hl", q[b].float(), ks) * scale
         out[b] = torch.einsum("hl,hld->hd", att.softmax(-1), vs).to(q.dtype)
     return out
+
+
+# ---------------------------------------------------------------------------------------------- hybrid layers
+def rmsnorm_f32(x, w, n, eps):
+    y = x * torch.rsqrt(x[:, :n].pow(2).mean(-1, keepdim=True) + eps)
+    return (y * w.float()).to(w.dtype)
+
+
+def softcap(z, cap):
+    return cap * torch.tanh(z / cap)
+
+
+def mamba2(p, m, wt, ring, state, batch, eps, out, out_pad, ff_col, ff):
+    """p fp32 [T, N]; see ``ops.hybrid.mamba2``."""
+    inner, cc, gn = m.inner, m.conv_channels, m.groups * m.state
+    rep = m.heads // m.groups
+    a = -wt.a_log.float().exp()
+    for i in range(batch.n):
+        t0, t1, start, row = int(batch.cu[i]), int(batch.cu[i + 1]), int(batch.start[i]), int(batch.row[i])
+        idle = batch.active is not None and int(batch.active[i]) == 0
+        u = p[t0:t1, inner:inner + cc]
+        past = [ring[row, (start - k) % m.conv].float() if start - k >= 0 else torch.zeros(cc)
+                for k in range(m.conv - 1, 0, -1)]
+        ext = torch.cat([torch.stack(past), u]) if past else u
+        conv = F.conv1d(ext.t()[None], wt.conv.float()[:, None], wt.conv_bias.float(), groups=cc)[0].t()
+        xbc = F.silu(conv).to(out.dtype).float()
+        dt = F.softplus(p[t0:t1, inner + cc:inner + cc + m.heads] + wt.dt_bias.float(), threshold=30.0)
+        s = torch.zeros_like(state[row]) if start == 0 else state[row].clone()
+        x = xbc[:, :inner].view(-1, m.heads, m.vdim)
+        b = xbc[:, inner:inner + gn].view(-1, m.groups, m.state).repeat_interleave(rep, 1)
+        c = xbc[:, inner + gn:].view(-1, m.groups, m.state).repeat_interleave(rep, 1)
+        for t in range(t1 - t0):
+            s = (a * dt[t]).exp()[:, None, None] * s + dt[t][:, None, None] * b[t][:, :, None] * x[t][:, None, :]
+            y = torch.einsum("hnp,hn->hp", s, c[t]) + wt.d.float()[:, None] * x[t]
+            y = (y.reshape(-1).to(out.dtype).float() * F.silu(p[t0 + t, :inner])).view(m.norm_groups, -1)
+            y = (y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)).reshape(-1)
+            out[t0 + t, :inner] = (y * wt.norm.float()).to(out.dtype)
+        if not idle:
+            state[row] = s
+            for o in range(max(0, t1 - t0 - (m.conv - 1)), t1 - t0):
+                ring[row, (start + o) % m.conv] = u[o].to(ring.dtype)
+    out[:, out_pad:out_pad + ff] = F.relu(p[:, ff_col:ff_col + ff]).square().to(out.dtype)
+
+
+def window_attention(p, m, table, k_cache, v_cache, batch, out, out_pad, ff_col, ff, page):
+    """p fp32 [T, N]; see ``ops.hybrid.window_attention``."""
+    T, half = p.shape[0], m.rot_dims // 2
+
+    def turn(x):
+        if half == 0:
+            return x
+        cs = table[batch.pos.long()]
+        cos, sin = cs[:, None, :, 0], cs[:, None, :, 1]
+        u, v = x[..., :half], x[..., half:2 * half]
+        return torch.cat([u * cos - v * sin, v * cos + u * sin, x[..., 2 * half:]], -1)
+
+    nq, nk = m.heads * m.dim, m.kv_heads * m.dim
+    q = turn(p[:, :nq].view(T, m.heads, m.dim)).to(out.dtype).float()
+    slots = batch.slots.long()
+    if m.kv_from is None:
+        k_cache[slots, :, :m.dim] = turn(p[:, nq:nq + nk].view(T, m.kv_heads, m.dim)).to(k_cache.dtype)
+        v_cache[slots, :, :m.vdim] = p[:, nq + nk:nq + nk + m.kv_heads * m.vdim].view(T, m.kv_heads, m.vdim).to(v_cache.dtype)
+    rep = m.heads // m.kv_heads
+    for i in range(batch.n):
+        t0, t1, start = int(batch.cu[i]), int(batch.cu[i + 1]), int(batch.start[i])
+        last = start + t1 - t0
+        j = torch.arange(last)
+        at = batch.block_table[i].long()[j // page] * page + j % page
+        k = k_cache[at, :, :m.dim].float().repeat_interleave(rep, 1)
+        v = v_cache[at, :, :m.vdim].float().repeat_interleave(rep, 1)
+        s = torch.einsum("thd,jhd->htj", q[t0:t1], k) * m.scale
+        ii = torch.arange(start, last)[:, None]
+        seen = j[None] <= ii
+        if m.window is not None:
+            seen &= (ii - j[None] < m.window) | (j[None] < m.keep_first)
+        s = s.masked_fill(~seen, float("-inf"))
+        if m.sink:
+            s = torch.cat([s, torch.zeros(*s.shape[:2], 1)], -1)
+        w = s.softmax(-1)[..., :last]
+        out[t0:t1, :m.out_cols] = torch.einsum("htj,jhd->thd", w, v).reshape(t1 - t0, -1).to(out.dtype)
+    out[:, out_pad:out_pad + ff] = F.relu(p[:, ff_col:ff_col + ff]).square().to(out.dtype)

@@ -44,7 +44,7 @@ class PyBlockManager:
 def _native():
     from ..ops import _lib
 
-    if not os.path.exists(_lib.LIB_PATH):
+    if not os.path.exists(_lib.lib_path()):
         return None
     L = _lib.lib()
     L.b200_pool_create.restype = ctypes.c_void_p

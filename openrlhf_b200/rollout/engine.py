@@ -11,6 +11,10 @@ step for all rows is captured once per batch-size bucket as a CUDA graph (embedd
 RoPE+KV-write, paged tcgen05 attention, o-proj GEMM(+residual), RMSNorm, gate_up GEMM, SwiGLU, down GEMM(+residual)]
 x L -> RMSNorm -> lm_head GEMM -> sampler -> advance) and replayed per token; the host only intervenes every few steps
 to hand out KV pages and retire finished rows.
+
+Models whose layers differ (``models/hybrid.py``) bring their own step function, which runs any ragged batch: prompts,
+portions of prompts and single tokens side by side. The engine keeps their per-layer caches (``layer_cache.py``): paged
+keys and values, and recurrent state in one row per engine row. ``extend`` feeds given tokens instead of sampling.
 """
 from __future__ import annotations
 
@@ -22,13 +26,16 @@ from dataclasses import dataclass, field
 import torch
 
 from ..models.config import ModelConfig
+from ..models.hybrid import HybridLM
 from ..models.transformer import TransformerLM
 from ..ops import _lib
 from ..ops import functional as F
 from ..ops.attention import PAGE, paged_decode, rope_kvwrite
-from ..ops.gemm import gemm, gemm_swiglu, swiglu_fusable
+from ..ops.gemm import decode_gemm, gemm, gemm_swiglu, gemm_to_workspace, swiglu_fusable
+from ..ops.hybrid import StepBatch
 from ..ops.sampling import sample
 from .block_manager import BlockManager
+from .layer_cache import LayerCache
 
 
 import os as _os
@@ -105,13 +112,21 @@ class _Pending:
 
 
 class RolloutEngine:
-    def __init__(self, model: TransformerLM, max_num_seqs: int = 256, max_model_len: int = 4096,
+    def __init__(self, model: TransformerLM | HybridLM, max_num_seqs: int = 256, max_model_len: int = 4096,
                  num_pages: int | None = None, gpu_memory_utilization: float = 0.5, seed: int = 0,
                  eos_token_id: int | None = None, use_cuda_graph: bool = True, check_interval: int = 16, tp=None,
                  quantization: str | None = None, enable_prefix_caching: bool = False,
                  max_prefill_tokens: int = 16384, decode_pdl: bool = False):
-        assert model.cfg.head_dim == 128 or not model.flat.is_cuda, \
-            "the decode attention kernel is specialised for head_dim 128"
+        self.hybrid = isinstance(model, HybridLM)
+        if self.hybrid:
+            if tp is not None or quantization is not None:
+                raise ValueError("hybrid models run in bf16 or fp32 on one GPU (no tensor parallelism, no quantisation)")
+            if enable_prefix_caching and model.cfg.has_recurrent_state:
+                raise ValueError("prefix caching needs the keys and values of a prefix to stand for it; recurrent state "
+                                 "does not live in pages")
+        else:
+            assert model.cfg.head_dim == 128 or not model.flat.is_cuda, \
+                "the decode attention kernel is specialised for head_dim 128"
         assert quantization in (None, "fp8"), "rollout quantisation: None or 'fp8' (per-tensor e4m3)"
         self.model = model
         # fp8 decode: the projection weights are kept as e4m3 copies with one scale per matrix (re-quantised after
@@ -135,17 +150,24 @@ class RolloutEngine:
         self.use_cuda_graph = use_cuda_graph and self.on_gpu
         self.check_interval = check_interval
         cfg = self.cfg
-        bytes_per_page = 2 * cfg.num_hidden_layers * PAGE * cfg.kv_size * 2
+        row_bytes = 0
+        if self.hybrid:
+            specs = model.cache_specs()
+            bytes_per_page = max(1, LayerCache.bytes_per(specs, "page", PAGE))
+            row_bytes = LayerCache.bytes_per(specs, "row", PAGE)
+        else:
+            bytes_per_page = 2 * cfg.num_hidden_layers * PAGE * cfg.kv_size * 2
         if num_pages is None and not self.on_gpu:
             num_pages = max(8, min(max_num_seqs * self.max_pages + 1, 2048))
         if num_pages is None:
             free, total = torch.cuda.mem_get_info(self.device)
-            budget = int(total * gpu_memory_utilization) - (total - free)
+            budget = int(total * gpu_memory_utilization) - (total - free) - max_num_seqs * row_bytes
             num_pages = max(8, min(budget // bytes_per_page, max_num_seqs * self.max_pages + 1))
         self.num_pages = int(num_pages)
         self.blocks = BlockManager(self.num_pages)
         self.dummy_page = self.blocks.alloc()  # page 0 backs inactive rows
         self.kv = None
+        self.cache: LayerCache | None = None
         self.arena = None
         self._alloc_kv()
         B = max_num_seqs
@@ -175,8 +197,10 @@ class RolloutEngine:
         self.max_new_cap = max_model_len
         self.out_tokens = torch.zeros(B, self.max_new_cap, dtype=torch.int64, device=dev)
         self.out_logprobs = torch.zeros(B, self.max_new_cap, dtype=torch.float32, device=dev)
-        self.q_buf = torch.empty(B, cfg.num_attention_heads, cfg.head_dim, dtype=model.flat.dtype, device=dev)
-        self.attn_buf = torch.empty_like(self.q_buf)
+        if not self.hybrid:
+            self.q_buf = torch.empty(B, cfg.num_attention_heads, cfg.head_dim, dtype=model.flat.dtype, device=dev)
+            self.attn_buf = torch.empty_like(self.q_buf)
+        self.row_ids = torch.arange(B + 1, dtype=torch.int32, device=dev)    # state row of every engine row
         self.next_tok = torch.zeros(B, dtype=torch.int64, device=dev)
         self.next_lp = torch.zeros(B, dtype=torch.float32, device=dev)
         self.rows: list[_Row | None] = [None] * B
@@ -187,6 +211,7 @@ class RolloutEngine:
         self._table_dirty = False
         self._stale_rows: list = []
         self._req: dict = {}
+        self._sessions: dict = {}               # requests driven token by token through extend(): key -> row
         self._batch_counter = 0
         self.graphs: dict[tuple, torch.cuda.CUDAGraph] = {}
         self.graph_launches: dict[tuple, int] = {}
@@ -206,33 +231,42 @@ class RolloutEngine:
         self.stats = {"preemptions": 0, "prefix_hit_tokens": 0, "prefill_tokens": 0, "prefill_chunks": 0}
         if self.on_gpu:
             _lib.status_word(self.device)
-        self.model.rope(self.device)
+        if self.hybrid:
+            self.model.ensure_positions(max_model_len)
+        else:
+            self.model.rope(self.device)
 
     # ------------------------------------------------------------------ memory
     def _alloc_kv(self):
         """KV cache [layers, 2, pages*128, kv_heads, 128] inside a VMM arena: its address survives sleep / wake."""
+        if self.hybrid:
+            if self.cache is None:
+                self.cache = LayerCache(self.model.cache_specs(), self.num_pages, PAGE, self.max_num_seqs, self.device)
+            self.cache.bind(self._arena_bytes(self.cache.nbytes) if self.on_gpu else
+                            torch.zeros(self.cache.nbytes, dtype=torch.uint8))
+            return
         cfg = self.cfg
         shape = (cfg.num_hidden_layers, 2, self.num_pages * PAGE, cfg.num_key_value_heads, cfg.head_dim)
         if not self.on_gpu:
             self.kv = torch.zeros(*shape, dtype=self.model.flat.dtype, device=self.device)
             return
-        if getattr(self, "arena", None) is None:
+        nbytes = 2 * math.prod(shape)
+        self.kv = self._arena_bytes(nbytes)[:nbytes].view(torch.bfloat16).view(*shape)
+        self.kv.zero_()           # stale V rows are multiplied by zero probabilities: they must be finite
+
+    def _arena_bytes(self, nbytes: int) -> torch.Tensor:
+        """uint8 buffer for the caches: the VMM arena (mapped again after a sleep), or a plain allocation where the
+        driver has no VMM support (captured graphs are then dropped on sleep)."""
+        if self.arena is None:
             try:
                 from .block_manager import VmmArena
 
-                nbytes = 2
-                for d in shape:
-                    nbytes *= d
                 self.arena = VmmArena(nbytes, self.device)
-            except Exception:  # noqa: BLE001  (driver without VMM support: plain allocation, graphs dropped on sleep)
-                self.arena = None
-        if self.arena is not None:
-            if not self.arena.mapped:
-                self.arena.map()
-            self.kv = self.arena.tensor(torch.bfloat16, shape)
-            self.kv.zero_()       # stale V rows are multiplied by zero probabilities: they must be finite
-        else:
-            self.kv = torch.zeros(*shape, dtype=torch.bfloat16, device=self.device)
+            except Exception:  # noqa: BLE001
+                return torch.empty(nbytes, dtype=torch.uint8, device=self.device)
+        if not self.arena.mapped:
+            self.arena.map()
+        return self.arena.tensor(torch.uint8, (nbytes,))
 
     def sleep(self, level: int = 1):
         """Release the physical memory of the KV cache. Weights stay resident: trainer and rollout share them on this
@@ -245,6 +279,8 @@ class RolloutEngine:
         else:
             self.graphs.clear()
             self.kv = None
+            if self.cache is not None:
+                self.cache.release()
             if self.on_gpu:
                 torch.cuda.empty_cache()
         self.sleeping = True
@@ -307,17 +343,57 @@ class RolloutEngine:
     # ------------------------------------------------------------------ model execution
     @torch.no_grad()
     def _prefill(self, items: list, mms: list | None = None):
-        """Run one prefill pass. items: list of (tokens, start, row) where `tokens` is the whole context of the row so
-        far (prompt, plus generated tokens of a preempted sample), `start` the number of leading tokens whose KV already
-        sits in the row's pages (prefix-cache hit or earlier chunks) and the rest, tokens[start:], is computed now and
-        written to the pages of `row`. Returns the logits [len(items), V] at the last position of every item.
+        """One prefill pass over (context so far, number of its leading tokens whose state is cached, row): the rest of
+        every context is computed. Returns the logits [len(items), V] at the last position of every item."""
+        return self._forward_tokens([(t[s0:], s0, row, [len(t) - s0 - 1]) for t, s0, row in items], mms)
+
+    def _ragged_batch(self, items: list) -> StepBatch:
+        """Step descriptor of items (new tokens, start, row, ...), built on the host and copied in one transfer."""
+        lens = [len(it[0]) for it in items]
+        starts = [it[1] for it in items]
+        n, T = len(items), sum(lens)
+        pos = torch.cat([torch.arange(s0, s0 + k, dtype=torch.int32) for s0, k in zip(starts, lens)])
+        tok_seq = torch.repeat_interleave(torch.arange(n, dtype=torch.int32), torch.tensor(lens))
+        pages = torch.full((n, max(len(self.rows[it[2]].pages) for it in items)), self.dummy_page, dtype=torch.int32)
+        for i, it in enumerate(items):
+            pg = self.rows[it[2]].pages
+            pages[i, :len(pg)] = torch.tensor(pg, dtype=torch.int32)
+        slots = pages[tok_seq.long(), (pos // PAGE).long()] * PAGE + pos % PAGE
+        cu = torch.zeros(n + 1, dtype=torch.int32)
+        cu[1:] = torch.cumsum(torch.tensor(lens), 0)
+        parts = [torch.tensor([x for it in items for x in it[0]], dtype=torch.int32), pos, slots, tok_seq, cu,
+                 torch.tensor(starts, dtype=torch.int32), torch.tensor([it[2] for it in items], dtype=torch.int32),
+                 pages.reshape(-1)]
+        flat = torch.cat([torch.nn.functional.pad(p, (0, -p.numel() % 4)) for p in parts]).to(self.device)   # 16 B apart
+        out, o = [], 0
+        for p in parts:
+            out.append(flat[o:o + p.numel()])
+            o += (p.numel() + 3) // 4 * 4
+        return StepBatch(out[0].long(), out[1], out[2], out[3], out[4], out[5], out[6], out[7].view(n, -1), n, T, max(lens))
+
+    @torch.no_grad()
+    def _forward_tokens(self, items: list, mms: list | None = None):
+        """Run tokens of several sequences as one batch. items: list of (new tokens, start, row, want): the sequence of
+        `row` already holds `start` tokens (earlier chunks, a prefix-cache hit, decoded tokens); the new ones are
+        computed and written to the row's pages and state. Returns the logits at the wanted places (indices into the new
+        tokens), in the order of the items; None when nothing is wanted.
         mms: per item None or {"pixel_values", "image_grid_thw"} (only with start == 0); sets the rotary offsets."""
+        if self.hybrid:
+            batch = self._ragged_batch(items)
+            offs, o = [], 0
+            for it in items:
+                offs += [o + k for k in it[3]]
+                o += len(it[0])
+            self.stats["prefill_tokens"] += batch.T
+            self.stats["prefill_chunks"] += 1
+            want = None if offs == list(range(batch.T)) else torch.tensor(offs, dtype=torch.int32, device=self.device)
+            return self.model.step(batch, self.cache, want)
         cfg, m = self.cfg, self.model
         dev = self.device
         n_items = len(items)
-        new_lens = [len(t) - s0 for t, s0, _ in items]
-        starts = [s0 for _, s0, _ in items]
-        ids = torch.tensor([x for t, s0, _ in items for x in t[s0:]], dtype=torch.int64, device=dev)
+        new_lens = [len(it[0]) for it in items]
+        starts = [it[1] for it in items]
+        ids = torch.tensor([x for it in items for x in it[0]], dtype=torch.int64, device=dev)
         pos = torch.cat([torch.arange(s0, s0 + n, dtype=torch.int32) for s0, n in zip(starts, new_lens)]).to(dev)
         cu_new = [0]
         for n in new_lens:
@@ -328,16 +404,15 @@ class RolloutEngine:
             pages = self.rows[row].pages
             return [pages[t // PAGE] * PAGE + t % PAGE for t in range(a, b)]
 
-        slots = torch.tensor([x for (t, s0, row) in items for x in slots_of(row, s0, len(t))], dtype=torch.int64,
+        slots = torch.tensor([x for it in items for x in slots_of(it[2], it[1], it[1] + len(it[0]))], dtype=torch.int64,
                              device=dev)
         with_prefix = any(starts)
         if with_prefix:
             # rows of the full (prefix + new) stream: where each sequence's cached keys live, and where the new ones go
             cu_all = [0]
-            for t, _, _ in items:
-                cu_all.append(cu_all[-1] + len(t))
-            pre_slots = torch.tensor([x for (t, s0, row) in items for x in slots_of(row, 0, s0)], dtype=torch.int64,
-                                     device=dev)
+            for it in items:
+                cu_all.append(cu_all[-1] + it[1] + len(it[0]))
+            pre_slots = torch.tensor([x for it in items for x in slots_of(it[2], 0, it[1])], dtype=torch.int64, device=dev)
             pre_rows = torch.cat([torch.arange(cu_all[i], cu_all[i] + starts[i]) for i in range(n_items)]).to(dev)
             new_rows = torch.cat([torch.arange(cu_all[i] + starts[i], cu_all[i + 1]) for i in range(n_items)]).to(dev)
             scale = 1.0 / math.sqrt(cfg.head_dim)
@@ -370,12 +445,12 @@ class RolloutEngine:
                 thw = torch.cat([torch.as_tensor(mm["image_grid_thw"]).view(-1, 3) for mm in mms if mm])
                 embeds, pos = m.multimodal_inputs(ids, cu_new, pv, thw)
                 merge = cfg.vision_config().spatial_merge_size
-                for k_, ((t, _, _), mm) in enumerate(zip(items, mms)):
+                for k_, ((t, _, _, _), mm) in enumerate(zip(items, mms)):
                     if mm:
                         grids = [tuple(g) for g in torch.as_tensor(mm["image_grid_thw"]).view(-1, 3).tolist()]
                         deltas[k_] = mrope_positions(t, grids, cfg.image_token_id, merge, cfg.video_token_id)[1]
-            for d, (_, _, row) in zip(deltas, items):
-                self.rope_delta[row] = d
+            for d, it in zip(deltas, items):
+                self.rope_delta[it[2]] = d
         # ranks prefill independently of each other: expert-parallel dispatch (a collective of the training passes) is
         # off here, every rank runs all experts of its own copy of the weights
         ep_saved, m.ep = m.ep, None
@@ -384,13 +459,19 @@ class RolloutEngine:
         finally:
             m.ep = ep_saved
         m.train(was_training)
-        last = (cu[1:] - 1).long()
+        rows = torch.tensor([c + k for c, it in zip(cu_new, items) for k in it[3]], dtype=torch.int64, device=dev)
         self.stats["prefill_tokens"] += int(cu_new[-1])
         self.stats["prefill_chunks"] += 1
-        return F.linear(h[last].contiguous(), m.lm_head_weight())
+        if rows.numel() == 0:
+            return None
+        return F.linear(h[rows].contiguous(), m.lm_head_weight())
 
     def _decode_step(self, B: int):
         """One token for rows [0, B). Pure device work on static buffers: safe to capture in a CUDA graph."""
+        if self.hybrid:
+            logits = self.model.step(self._decode_batch(B), self.cache)
+            self._sample_rows(logits, B)
+            return
         cfg, m = self.cfg, self.model
         fused = (not cfg.qk_norm and cfg.num_experts == 0 and m.lora is None and self.quantization is None
                  and self.on_gpu)
@@ -404,6 +485,15 @@ class RolloutEngine:
                 logits = self._decode_layers_fused(B)
         else:
             logits = self._decode_layers_generic(B)
+        self._sample_rows(logits, B)
+
+    def _decode_batch(self, B: int) -> StepBatch:
+        """The rows [0, B) as a batch of single tokens over the engine's static buffers."""
+        ids = self.row_ids
+        return StepBatch(self.tok[:B], self.pos[:B], self.slots[:B], ids[:B], ids[:B + 1], self.pos[:B], ids[:B],
+                         self.block_table[:B], B, B, 1, active=self.active[:B])
+
+    def _sample_rows(self, logits: torch.Tensor, B: int):
         sample(logits, temperature=self.temperature[:B], top_k=self.top_k_rows[:B], top_p=self.top_p_rows[:B], seed=self.seed,
                step=self.step_counter, out_tokens=self.next_tok[:B], out_logprobs=self.next_lp[:B],
                active=self.active[:B])
@@ -566,6 +656,8 @@ class RolloutEngine:
         if g is None:
             # warm up outside capture (lazy library state, status word, rope table), then capture
             saved = self._snapshot_state(B)
+            if self.hybrid:
+                self.active.zero_()          # the warm-up step must leave the recurrent state alone
             s = torch.cuda.Stream(device=self.device)
             s.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(s):
@@ -982,6 +1074,51 @@ class RolloutEngine:
             outs.append(ro)
         return outs
 
+    # ------------------------------------------------------------------ given tokens instead of sampled ones
+    @torch.no_grad()
+    def extend(self, entries: list) -> torch.Tensor | None:
+        """Feed given tokens: entries is a list of (key, new token ids, wanted places among them). All entries run as one
+        batch, from the cache and state that earlier calls left; a key that is not live yet is admitted. Returns the
+        fp32 logits at the wanted places, in order, or None. ``finish`` gives back what a key holds.
+
+        A batch of single tokens of live sequences takes the decode kernels, everything else the ragged ones, as when
+        the engine generates."""
+        entries = [e for e in entries if len(e[1])]
+        if not entries:
+            return None
+        if self.sleeping:
+            self.wake_up()
+        assert len({e[0] for e in entries}) == len(entries), "a sequence can bring only one portion per step"
+        items = []
+        for key, tokens, want in entries:
+            row = self._sessions.get(key)
+            if row is None:
+                row = next((i for i, r in enumerate(self.rows) if r is None), None)
+                if row is None:
+                    raise RuntimeError("no free row: finish a sequence first")
+                self._order += 1
+                self.rows[row] = _Row(key, 0, 0, 0, [], order=self._order, prefilled=0)
+                self.block_table_host[row].fill_(self.dummy_page)
+                self._sessions[key] = row
+            r = self.rows[row]
+            end = r.prefilled + len(tokens)
+            if end > self.max_model_len:
+                raise ValueError(f"sequence {key!r} would hold {end} tokens, max_model_len is {self.max_model_len}")
+            if self._pages_short(row, end - 1) > self._free_pages():
+                raise RuntimeError("the KV cache is full: finish a sequence first")
+            self._ensure_pages(row, end - 1)
+            items.append((list(tokens), r.prefilled, row, list(want)))
+        logits = self._forward_tokens(items)
+        for (tokens, _, row, _) in items:
+            self.rows[row].prefilled += len(tokens)
+        if self.on_gpu:
+            _lib.check_status(self.device)
+        return None if logits is None else logits.float()
+
+    def finish(self, key) -> None:
+        """Release the row, pages and state of a sequence that was fed through ``extend``."""
+        self._release_row(self._sessions.pop(key))
+
     def _start_rows(self, logits: torch.Tensor, entries: list):
         """Contexts whose prefill is complete: copy the open page to the other samples of each request, draw the first
         token of every row from the last-position logits and initialise the rows' device state."""
@@ -997,7 +1134,12 @@ class RolloutEngine:
                 src = self.rows[rows[0]].pages[n_full]
                 for r in rows[1:]:
                     dst = self.rows[r].pages[n_full]
-                    self.kv[:, :, dst * PAGE:(dst + 1) * PAGE].copy_(self.kv[:, :, src * PAGE:(src + 1) * PAGE])
+                    if self.hybrid:
+                        self.cache.copy_page(src, dst)
+                    else:
+                        self.kv[:, :, dst * PAGE:(dst + 1) * PAGE].copy_(self.kv[:, :, src * PAGE:(src + 1) * PAGE])
+            if self.hybrid and len(rows) > 1:
+                self.cache.copy_row(rows[0], rows[1:])
             if self.mrope and len(rows) > 1:
                 self.rope_delta[rows[1:]] = self.rope_delta[rows[0]]
         rep = torch.tensor([len(g) for g in groups], device=dev)
@@ -1042,51 +1184,3 @@ class RolloutEngine:
             for r in g:
                 self.rows[r].gen = self.rows[r].base + 1
                 self.rows[r].prefilled = -1
-
-
-# ---------------------------------------------------------------------------------------------- decode GEMM
-_BN64_MAX_N = 2048      # widest output for which 64-column tiles (more CTAs) beat 128-column tiles at short K
-
-
-def gemm_to_workspace(x: torch.Tensor, w: torch.Tensor, ws: torch.Tensor | None = None):
-    """Split-K projection for small M whose fp32 slabs stay in the shared workspace for the next kernel to reduce.
-    Returns (workspace, number of slabs). `ws`: use this buffer (a symmetric one under tensor parallelism)."""
-    from ..ops.gemm import splitk_workspace
-
-    M, K = x.shape
-    N = w.shape[0]
-    # narrow N tiles give more CTAs for short K; with a long K (down_proj) 128-wide tiles halve the activation re-reads
-    # per weight byte and twice as many K splits keep all SMs streaming (14.4 us vs 16.9 us at N 1536, K 8960)
-    bn = 64 if (N <= _BN64_MAX_N and K < 4096) else 128      # small matrices only (e.g. 1536 x 1536): more CTAs
-    tiles = ((M + 127) // 128) * ((N + bn - 1) // bn)
-    kb = (K + 63) // 64
-    splits = max(1, min(148 // max(tiles, 1), kb // 4))
-    per = (kb + splits - 1) // splits
-    splits = (kb + per - 1) // per
-    if ws is None:
-        ws = splitk_workspace(x.device, splits * M * N)
-    assert ws.numel() >= splits * M * N
-    gemm(x, w, out=ws, k_splits=splits, split_stride=M * N, bn=bn)
-    return ws, splits
-
-
-
-
-def decode_gemm(x: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None = None,
-                residual: torch.Tensor | None = None) -> torch.Tensor:
-    """Small-M linear for the decode loop: picks a narrow N tile and split-K so that all SMs stream weights."""
-    from ..ops.gemm import gemm_splitk
-
-    M, K = x.shape
-    N = w.shape[0]
-    if not x.is_cuda:
-        return F.linear(x, w, bias, residual)
-    if M > 256:
-        return gemm(x, w, bias=bias, residual=residual)
-    bn = 64 if (N <= _BN64_MAX_N and K < 4096) else 128
-    tiles = ((M + 127) // 128) * ((N + bn - 1) // bn)
-    kb = (K + 63) // 64
-    splits = max(1, min(148 // max(tiles, 1), kb // 4))
-    if splits <= 1:
-        return gemm(x, w, bias=bias, residual=residual, bn=bn)
-    return gemm_splitk(x, w, splits, bias=bias, residual=residual, bn=bn)

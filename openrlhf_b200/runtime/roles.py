@@ -15,6 +15,7 @@ import torch
 import torch.distributed as dist
 
 from ..models.hf_io import load_pretrained
+from ..models.registry import read_config, require_trainable
 from ..parallel.zero import LRScheduler, ZeroEngine
 
 
@@ -38,6 +39,7 @@ def build_trainable(strategy, path: str, node: SimpleNamespace, *, device, max_s
     engine needs a copy of its own refreshed by the gather kernel; ("tp_train", model) - tensor-parallel shards."""
     a = strategy.args
     zw = strategy.zero_world
+    require_trainable(read_config(path))
     lm = load_pretrained(path, device=device, with_lm_head=with_lm_head, with_value_head=with_value_head,
                          shard_world=zw, seed=seed, value_head_prefix=value_head_prefix)
     tp_train = strategy.ds_tensor_parallel_size > 1 and strategy.world_size > 1
