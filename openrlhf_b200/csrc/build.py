@@ -29,11 +29,11 @@ NVCC_FLAGS = [
 ]
 
 # no fast-math: these kernels carry 32-bit recurrences, norms and logits and name their fast intrinsics one by one
-PRECISE = {"hybrid_ops.cu", "ssd.cu", "attn_window.cu", "gemm_f32.cu"}
+PRECISE = {"hybrid_ops.cu", "ssd.cu", "ssd_chunk.cu", "attn_window.cu", "gemm_f32.cu"}
 
 COMPONENTS = {
     "serve_hybrid": ["gemm_tcgen05.cu", "gemm2_tcgen05.cu", "elementwise.cu", "sampling.cu", "host_runtime.cu",
-                     "hybrid_ops.cu", "ssd.cu", "attn_window.cu", "attn_decode.cu", "gemm_f32.cu"],
+                     "hybrid_ops.cu", "ssd.cu", "ssd_chunk.cu", "attn_window.cu", "attn_decode.cu", "gemm_f32.cu"],
 }
 
 

@@ -51,7 +51,7 @@ conv_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, const
     const int t = (int)(idx / per_tok), e = (int)(idx % per_tok);
     if (e >= nv) {
       const int h = e - nv;
-      dt[(size_t)t * d.H + h] = softplus_f(src.get_raw(t, d.inner + d.cc + h) + to_f(dt_bias[h]));
+      dt[(size_t)h * b.T + t] = softplus_f(src.get_raw(t, d.inner + d.cc + h) + to_f(dt_bias[h]));
       continue;
     }
     const int c = e * V;
@@ -116,7 +116,7 @@ ssd_scan_kernel(const T* __restrict__ xbc, const float* __restrict__ dt, const R
       sc[k] = to_f(r[d.inner + (d.G + g) * d.N + k]);
     }
     for (int k = threadIdx.x; k < d.P; k += blockDim.x) sx[k] = to_f(r[h * d.P + k]);
-    const float dtv = dt[(size_t)(row0 + o) * d.H + h];
+    const float dtv = dt[(size_t)h * b.T + row0 + o];
     const float decay = expf(a * dtv);
     __syncthreads();
     if (pg < ng) {
@@ -245,7 +245,7 @@ static int launch_conv(const Proj<T>& src, const Ragged& b, T* ring, const T* w,
 using namespace b200;
 #define SSD_STREAM(s) reinterpret_cast<cudaStream_t>(s)
 
-// Causal convolution + silu of a ragged batch, step sizes, and the ring update. out [T, cc], dt fp32 [T, H].
+// Causal convolution + silu of a ragged batch, step sizes, and the ring update. out [T, cc], dt fp32 [H, T].
 extern "C" int b200_ssd_conv(const void* p, const float* ws, int splits, long long slab, int ld, const int* cu,
                              const int* start, const int* row, const int* active, const int* tok_seq, int n, int T,
                              void* ring, const void* w, const void* bias, const void* dt_bias, void* out, float* dt, int H,

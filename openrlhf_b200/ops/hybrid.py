@@ -159,6 +159,28 @@ class Mamba2Weights:
     norm: torch.Tensor       # [inner]
 
 
+CHUNK_MIN = 8      # portions of at least this many tokens take the tensor-core scan
+
+
+def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, m, a_log: torch.Tensor, d: torch.Tensor, state: torch.Tensor,
+             y: torch.Tensor, batch: StepBatch, chunked: bool | None = None) -> None:
+    """Recurrence over the convolved inputs xbc [T, channels] and step sizes dt fp32 [heads, T]; y [T, inner]. `chunked`
+    picks the tensor-core kernel (bf16, sizes it covers) or the token-by-token one; None: by portion length."""
+    L = _lib.lib()
+    seqs = (_p(batch.cu), _p(batch.start), _p(batch.row), _p(batch.active), _p(batch.tok_seq), _i(batch.n), _i(batch.T))
+    H, P, N, G = _i(m.heads), _i(m.vdim), _i(m.state), _i(m.groups)
+    fits = xbc.dtype == torch.bfloat16 and L.b200_ssd_chunk_fits(H, P, N, G) == 1
+    if chunked is None:
+        chunked = fits and batch.max_new >= CHUNK_MIN
+    if chunked:
+        assert fits, "sizes outside the tensor-core scan"
+        _lib.check_rc(L.b200_ssd_chunk(_p(xbc), _p(dt), *seqs, _p(a_log), _p(d), _p(state), _p(y), H, P, N, G,
+                                       _p(_lib.status_word(xbc.device)), _lib.stream_ptr()), "ssd_chunk")
+    else:
+        _lib.check_rc(L.b200_ssd_scan(_p(xbc), _p(dt), *seqs, _p(a_log), _p(d), _p(state), _p(y), H, P, N, G, _i(m.conv),
+                                      _f32(xbc.dtype), _lib.stream_ptr()), "ssd_scan")
+
+
 def mamba2(p: Projection, m, wt: Mamba2Weights, ring: torch.Tensor, state: torch.Tensor, batch: StepBatch, eps: float,
            out: torch.Tensor, out_pad: int, ff_col: int, ff: int) -> None:
     """Convolution, recurrence, gate and group norm of one layer: columns [0, inner) of `out` [T, ld]; the feed-forward
@@ -179,11 +201,10 @@ def mamba2(p: Projection, m, wt: Mamba2Weights, ring: torch.Tensor, state: torch
     else:
         seqs = (_p(batch.cu), _p(batch.start), _p(batch.row), _p(batch.active), _p(batch.tok_seq), _i(batch.n), _i(T))
         xbc = torch.empty(T, m.conv_channels, dtype=p.dtype, device=dev)
-        dt = torch.empty(T, m.heads, dtype=torch.float32, device=dev)
+        dt = torch.empty(m.heads, T, dtype=torch.float32, device=dev)
         _lib.check_rc(L.b200_ssd_conv(*p.args(), *seqs, _p(ring), _p(wt.conv), _p(wt.conv_bias), _p(wt.dt_bias), _p(xbc),
                                       _p(dt), *dims, f32, st()), "ssd_conv")
-        _lib.check_rc(L.b200_ssd_scan(_p(xbc), _p(dt), *seqs, _p(wt.a_log), _p(wt.d), _p(state), _p(y), *dims, f32, st()),
-                      "ssd_scan")
+        ssd_scan(xbc, dt, m, wt.a_log, wt.d, state, y, batch)
     _lib.check_rc(L.b200_gate_norm(_p(y), *p.args(), _p(wt.norm), _p(out), _i(out.stride(0)), _i(T), _i(m.inner),
                                    _i(m.norm_groups), _f(eps), _i(ff_col), _i(ff), _p(out[:, out_pad:]), f32, st()),
                   "gate_norm")
