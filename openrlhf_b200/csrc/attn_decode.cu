@@ -27,6 +27,22 @@ struct DecodeParams {
   float scale_log2;        // softmax scale * log2(e)
   int* status;
   int early_trigger;       // the grid fits in one wave (two CTAs per SM): dependents may be released at once
+  // windowed variant: head sizes up to 128 through 3-D tensor maps (channels past dk / dv read as zero), a window that
+  // keeps the first tokens, a sink of score 0, a free output row stride
+  int len_add;             // tokens in the cache = seq_lens[b] + len_add
+  int window, keep, sink;
+  int dk, dv, out_ld;
+};
+
+// Pages a query at the end of `len` tokens reads: those with kept first tokens, then those of the window.
+struct PageList {
+  int kept, w0, n;
+  __device__ __forceinline__ PageList(int len, int window, int keep) {
+    w0 = max(0, len - window) / PAGE;
+    kept = min((keep + PAGE - 1) / PAGE, w0);
+    n = kept + (len - 1) / PAGE - w0 + 1;
+  }
+  __device__ __forceinline__ int page(int t) const { return t < kept ? t : w0 + (t - kept); }
 };
 
 struct DecSmem {
@@ -43,6 +59,8 @@ struct DecSmem {
 // double-buffered (TMEM columns [0,16) / [16,32), shared-memory P buffers 0 / 1). The running output O (TMEM
 // columns [32,48)) is rescaled only when a head's maximum grew by more than 2^8 since the reference maximum was
 // last moved, which needs the previous P*V to have finished (pv_done); otherwise nothing waits on the tensor pipe.
+// WIN: the windowed variant (DecodeParams).
+template <bool WIN>
 __global__ void __launch_bounds__(192, 2)
 attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                    const __grid_constant__ CUtensorMap tma_v, const DecodeParams p) {
@@ -96,8 +114,10 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
   const uint32_t tmem_o = tmem_base + 32;   // 16 columns
   if (p.early_trigger) pdl_launch_dependents();
   pdl_wait();   // seq_lens / block_table / q / the KV cache come from earlier kernels of the stream
-  const int len = p.seq_lens[b];
-  const int n_tiles_all = (len + PAGE - 1) / PAGE;
+  const int len = WIN ? p.seq_lens[b] + p.len_add : p.seq_lens[b];
+  const PageList pages(len, WIN ? p.window : 1 << 30, WIN ? p.keep : 0);
+  const int n_tiles_all = WIN ? pages.n : (len + PAGE - 1) / PAGE;
+  const int kp = WIN ? (p.dk + 63) >> 6 : 2, vp = WIN ? (p.dv + 63) >> 6 : 2;      // 64-channel panels
   const int tiles_per_split = (n_tiles_all + p.splits - 1) / p.splits;
   const int tile0 = split * tiles_per_split;
   const int tile1 = min(n_tiles_all, tile0 + tiles_per_split);
@@ -110,22 +130,30 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
         tma_prefetch_desc(&tma_k);
         tma_prefetch_desc(&tma_v);
         // Q^T operand: 16 rows (heads of this kv group; rows beyond G are ignored) x 128 dims, two 64-wide panels
-        mbar_expect_tx(q_full, 2 * NPAD * 128);
+        mbar_expect_tx(q_full, kp * NPAD * 128);
         tma_load_2d(smem + DecSmem::Q_OFF, &tma_q, q_full, 0, b * p.Hq + kvh * G);
-        tma_load_2d(smem + DecSmem::Q_OFF + NPAD * 128, &tma_q, q_full, 64, b * p.Hq + kvh * G);
+        if (kp > 1) tma_load_2d(smem + DecSmem::Q_OFF + NPAD * 128, &tma_q, q_full, 64, b * p.Hq + kvh * G);
         uint8_t* sk = smem + DecSmem::K_OFF;
         uint8_t* sv = smem + DecSmem::V_OFF;
         uint32_t phase = 0;
         for (int t = tile0; t < tile1; ++t, phase ^= 1) {
-          const int page = p.block_table[(size_t)b * p.max_pages + t];
+          const int page = p.block_table[(size_t)b * p.max_pages + (WIN ? pages.page(t) : t)];
           if (!mbar_wait(k_empty, phase ^ 1, p.status, ERR_TIMEOUT_EMPTY)) break;
-          mbar_expect_tx(k_full, KV_TILE_BYTES);
-          tma_load_2d(sk, &tma_k, k_full, kvh * HD, page * PAGE);
-          tma_load_2d(sk + PAGE * 128, &tma_k, k_full, kvh * HD + 64, page * PAGE);
+          mbar_expect_tx(k_full, kp * (PAGE * 128));
+          if (WIN) {
+            for (int c = 0; c < kp; ++c) tma_load_3d(sk + c * PAGE * 128, &tma_k, k_full, c * 64, kvh, page * PAGE);
+          } else {
+            tma_load_2d(sk, &tma_k, k_full, kvh * HD, page * PAGE);
+            tma_load_2d(sk + PAGE * 128, &tma_k, k_full, kvh * HD + 64, page * PAGE);
+          }
           if (!mbar_wait(v_empty, phase ^ 1, p.status, ERR_TIMEOUT_EMPTY)) break;
-          mbar_expect_tx(v_full, KV_TILE_BYTES);
-          tma_load_2d(sv, &tma_v, v_full, kvh * HD, page * PAGE);
-          tma_load_2d(sv + PAGE * 128, &tma_v, v_full, kvh * HD + 64, page * PAGE);
+          mbar_expect_tx(v_full, vp * (PAGE * 128));
+          if (WIN) {
+            for (int c = 0; c < vp; ++c) tma_load_3d(sv + c * PAGE * 128, &tma_v, v_full, c * 64, kvh, page * PAGE);
+          } else {
+            tma_load_2d(sv, &tma_v, v_full, kvh * HD, page * PAGE);
+            tma_load_2d(sv + PAGE * 128, &tma_v, v_full, kvh * HD + 64, page * PAGE);
+          }
         }
       }
     } else if (warp == 1) {
@@ -144,7 +172,7 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
           for (int k = 0; k < HD / 16; ++k) {
             const uint64_t ad = make_smem_desc_sw128(sk + (k >> 2) * (PAGE * 128) + (k & 3) * 32, 16, 1024);
             const uint64_t bd = make_smem_desc_sw128(sq + (k >> 2) * (NPAD * 128) + (k & 3) * 32, 16, 1024);
-            umma_bf16(tmem_s + (j & 1) * NPAD, ad, bd, idesc_s, k > 0 ? 1u : 0u);
+            if (!WIN || k * 16 < p.dk) umma_bf16(tmem_s + (j & 1) * NPAD, ad, bd, idesc_s, k > 0 ? 1u : 0u);
           }
           umma_commit(&s_full[j & 1]);
           umma_commit(k_empty);          // the K buffer may be refilled as soon as these MMAs have read it
@@ -177,6 +205,10 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
       float m_ref[NPAD], l_part[NPAD];      // reference maximum (log2 domain) and this thread's share of the row sum
 #pragma unroll
       for (int h = 0; h < NPAD; ++h) { m_ref[h] = -INFINITY; l_part[h] = 0.f; }
+      if (WIN && p.sink && split == 0) {    // the sink's weight: score 0, counted by one thread of the first split
+#pragma unroll
+        for (int h = 0; h < NPAD; ++h) { m_ref[h] = 0.f; l_part[h] = row == 0 ? 1.f : 0.f; }
+      }
       bool ok = true;
       for (int i = 0; i < n_tiles && ok; ++i) {
         if (!mbar_wait(&s_full[i & 1], (i >> 1) & 1, p.status, ERR_TIMEOUT_TMEM_FULL)) { ok = false; break; }
@@ -184,7 +216,13 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
         uint32_t sr[NPAD];
         tmem_ld_32x32b_x16(tmem_s + (i & 1) * NPAD + lane_addr, sr);
         tmem_ld_wait();
-        const bool valid = (tile0 + i) * PAGE + row < len;
+        bool valid;
+        if (WIN) {
+          const int key = pages.page(tile0 + i) * PAGE + row;
+          valid = key < len && (key >= len - p.window || key < p.keep);
+        } else {
+          valid = (tile0 + i) * PAGE + row < len;
+        }
         float s[NPAD];
         float* redp = red + (i & 1) * 64;
 #pragma unroll
@@ -270,7 +308,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
             const float l = lred[h] + lred[NPAD + h] + lred[2 * NPAD + h] + lred[3 * NPAD + h];
             const float o = __uint_as_float(orr[h]) / l;
             if (p.splits == 1) {
-              p.out[((size_t)b * p.Hq + kvh * G + h) * HD + row] = __float2bfloat16_rn(o);
+              if (!WIN) p.out[((size_t)b * p.Hq + kvh * G + h) * HD + row] = __float2bfloat16_rn(o);
+              else if (row < p.dv) p.out[(size_t)b * p.out_ld + (kvh * G + h) * p.dv + row] = __float2bfloat16_rn(o);
             } else {
               const size_t idx = ((size_t)b * p.Hq + kvh * G + h) * p.splits + split;
               p.part_o[idx * HD + row] = o;
@@ -314,7 +353,8 @@ attn_decode_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
 
 // Merge split partials: out = sum_s w_s * o_s with w_s = l_s 2^(m_s - m) / sum(...)
 __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                         __nv_bfloat16* __restrict__ out, int rows /*B*Hq*/, int splits) {
+                                         __nv_bfloat16* __restrict__ out, int rows /*B*Hq*/, int splits, int Hq, int dv,
+                                         int out_ld) {
   const int r = blockIdx.x;
   const int d = threadIdx.x;
   if (r >= rows) return;
@@ -327,7 +367,7 @@ __global__ void attn_decode_merge_kernel(const float* __restrict__ part_o, const
     den += w;
     acc += w * part_o[((size_t)r * splits + s) * HD + d];
   }
-  out[(size_t)r * HD + d] = __float2bfloat16_rn(acc / den);
+  if (d < dv) out[(size_t)(r / Hq) * out_ld + (r % Hq) * dv + d] = __float2bfloat16_rn(acc / den);
 }
 
 // RoPE on q and k of freshly projected tokens + scatter of k, v into the paged cache + compact q output.
@@ -375,6 +415,8 @@ __global__ void rope_kvwrite_kernel(const __nv_bfloat16* __restrict__ qkv, const
 
 int make_tmap_bf16_2d(CUtensorMap* out, const void* base, uint64_t rows, uint64_t cols, uint64_t ld, uint32_t box_rows,
                       uint32_t box_cols);
+int make_tmap_bf16_3d(CUtensorMap* out, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t ld1, uint64_t ld2,
+                      uint32_t box0, uint32_t box1, uint32_t box2);
 
 }  // namespace b200
 
@@ -397,17 +439,54 @@ extern "C" int b200_attn_decode(const void* q, const void* k_cache, const void* 
   r = make_tmap_bf16_2d(&tv, v_cache, (uint64_t)num_pages * PAGE, (uint64_t)Hkv * HD, (uint64_t)Hkv * HD, PAGE, 64);
   if (r) return r;
   static std::atomic<unsigned long long> configured{0};      // one bit per device
-  if (!set_max_smem_once(configured, attn_decode_kernel, DecSmem::TOTAL)) return -2;
+  if (!set_max_smem_once(configured, attn_decode_kernel<false>, DecSmem::TOTAL)) return -2;
   DecodeParams p;
   p.block_table = block_table; p.seq_lens = seq_lens; p.out = reinterpret_cast<__nv_bfloat16*>(out);
   p.part_o = part_o; p.part_ml = part_ml; p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.max_pages = max_pages; p.splits = splits;
   p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
+  p.len_add = 0; p.window = 1 << 30; p.keep = 0; p.sink = 0; p.dk = HD; p.dv = HD; p.out_ld = Hq * HD;
   dim3 grid(Hkv, B, splits);
   p.early_trigger = (long long)Hkv * B * splits <= 2LL * 148 ? 1 : 0;      // two resident CTAs on each of 148 SMs
-  if (launch_pdl(attn_decode_kernel, grid, dim3(192), (size_t)DecSmem::TOTAL, stream, tq, tk, tv, p) != cudaSuccess) return -3;
+  if (launch_pdl(attn_decode_kernel<false>, grid, dim3(192), (size_t)DecSmem::TOTAL, stream, tq, tk, tv, p) != cudaSuccess) return -3;
   if (splits > 1) {
     attn_decode_merge_kernel<<<B * Hq, HD, 0, stream>>>(part_o, part_ml, reinterpret_cast<__nv_bfloat16*>(out), B * Hq,
-                                                        splits);
+                                                        splits, Hq, HD, Hq * HD);
+    if (cudaGetLastError() != cudaSuccess) return -3;
+  }
+  return 0;
+}
+
+// Windowed variant: q [B, H, dk_ld], caches [slots, G, dk_ld / dv_ld], tokens in the cache = pos[b] + 1 (the current one
+// included), out rows of out_ld elements with head h at column h * dv. Returns -20 for sizes it does not cover.
+extern "C" int b200_attn_decode_window(const void* q, const void* k_cache, const void* v_cache, const int* block_table,
+                                       const int* pos, void* out, int out_ld, float* part_o, float* part_ml, int B, int H,
+                                       int G, int dk, int dv, int dk_ld, int dv_ld, int num_pages, int max_pages, int splits,
+                                       int window, int keep, int sink, float scale, int* status, void* stream_) {
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  if (B <= 0) return 0;
+  if (H % G || splits < 1 || window < 1 || keep < 0) return -10;
+  if (H / G > NPAD || dk > HD || dv > HD || dk_ld % 8 || dv_ld % 8 || B > 65535) return -20;
+  if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) return -11;
+  CUtensorMap tq, tk, tv;
+  int r = make_tmap_bf16_2d(&tq, q, (uint64_t)B * H, dk, dk_ld, NPAD, 64);
+  if (r) return r;
+  r = make_tmap_bf16_3d(&tk, k_cache, dk, G, (uint64_t)num_pages * PAGE, dk_ld, (uint64_t)G * dk_ld, 64, 1, PAGE);
+  if (r) return r;
+  r = make_tmap_bf16_3d(&tv, v_cache, dv, G, (uint64_t)num_pages * PAGE, dv_ld, (uint64_t)G * dv_ld, 64, 1, PAGE);
+  if (r) return r;
+  static std::atomic<unsigned long long> configured{0};
+  if (!set_max_smem_once(configured, attn_decode_kernel<true>, DecSmem::TOTAL)) return -2;
+  DecodeParams p;
+  p.block_table = block_table; p.seq_lens = pos; p.out = reinterpret_cast<__nv_bfloat16*>(out);
+  p.part_o = part_o; p.part_ml = part_ml; p.B = B; p.Hq = H; p.Hkv = G; p.max_pages = max_pages; p.splits = splits;
+  p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
+  p.len_add = 1; p.window = window; p.keep = keep; p.sink = sink; p.dk = dk; p.dv = dv; p.out_ld = out_ld;
+  dim3 grid(G, B, splits);
+  p.early_trigger = (long long)G * B * splits <= 2LL * 148 ? 1 : 0;
+  if (launch_pdl(attn_decode_kernel<true>, grid, dim3(192), (size_t)DecSmem::TOTAL, stream, tq, tk, tv, p) != cudaSuccess) return -3;
+  if (splits > 1) {
+    attn_decode_merge_kernel<<<B * H, HD, 0, stream>>>(part_o, part_ml, reinterpret_cast<__nv_bfloat16*>(out), B * H,
+                                                       splits, H, dv, out_ld);
     if (cudaGetLastError() != cudaSuccess) return -3;
   }
   return 0;

@@ -33,7 +33,8 @@ PRECISE = {"hybrid_ops.cu", "ssd.cu", "ssd_chunk.cu", "attn_window.cu", "gemm_f3
 
 COMPONENTS = {
     "serve_hybrid": ["gemm_tcgen05.cu", "gemm2_tcgen05.cu", "elementwise.cu", "sampling.cu", "host_runtime.cu",
-                     "hybrid_ops.cu", "ssd.cu", "ssd_chunk.cu", "attn_window.cu", "attn_decode.cu", "gemm_f32.cu"],
+                     "hybrid_ops.cu", "ssd.cu", "ssd_chunk.cu", "attn_window.cu", "attn_window_tc.cu",
+                     "attn_decode.cu", "gemm_f32.cu"],
 }
 
 

@@ -7,7 +7,7 @@ scheduler tests."""
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 
 import torch
 
@@ -34,11 +34,23 @@ class StepBatch:
     T: int
     max_new: int                   # most tokens of one sequence in this step
     active: torch.Tensor | None = None    # [n] sequences with 0 leave every state as it is (idle rows of a decode bucket)
+    lens: list | None = None       # host copy of the portions' lengths (None: single tokens)
+    _tiles: dict = field(default_factory=dict)
 
     @property
     def single(self) -> bool:
         """Every sequence brings exactly one token."""
         return self.max_new == 1 and self.n == self.T
+
+    def query_tiles(self, tq: int):
+        """Query tiles of `tq` tokens: (sequence, first token inside the portion) of each, int32 on the device."""
+        hit = self._tiles.get(tq)
+        if hit is None:
+            lens = self.lens if self.lens is not None else [1] * self.n
+            pairs = torch.tensor([(i, q0) for i, k in enumerate(lens) for q0 in range(0, k, tq)], dtype=torch.int32)
+            pairs = pairs.t().contiguous().to(self.cu.device)
+            hit = self._tiles[tq] = (pairs[0], pairs[1], pairs.shape[1])
+        return hit
 
 
 @dataclass
@@ -243,9 +255,44 @@ def window_attention(p: Projection, m, table: torch.Tensor | None, k_cache: torc
         *p.args(), _p(batch.pos), _p(batch.slots), _p(table), _i(1 if table is None else table.shape[0]), _p(q), _p(k_cache),
         _p(v_cache), _i(T), _i(m.heads), _i(0 if m.kv_from is not None else m.kv_heads), _i(m.dim), _i(m.vdim), _i(m.k_ld),
         _i(m.v_ld), _i(m.rot_dims), _i(ff_col), _i(ff), _p(out[:, out_pad:]), _i(out.stride(0)), f32, st()), "rope_write")
+    attention(q, k_cache, v_cache, m, batch, out)
+
+
+def attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, m, batch: StepBatch, out: torch.Tensor,
+              impl: str | None = None) -> None:
+    """Attention of rotated queries q [T, heads, k_ld] over the paged cache. `impl`: "ragged" (any size and type),
+    "tiles" (tensor cores, bf16, heads up to 128 channels) or "decode" (the same for single tokens, groups of up to 16
+    query heads); None picks."""
+    L = _lib.lib()
     window = (1 << 30) if m.window is None else int(m.window)
+    rep = m.heads // m.kv_heads
+    fits = q.dtype == torch.bfloat16 and m.dim <= 128 and m.vdim <= 128 and rep <= 64
+    if impl is None:
+        impl = ("decode" if batch.single and rep <= 16 else "tiles") if fits else "ragged"
+    if impl == "decode":
+        # one CTA per (sequence, kv head, split): split the pages of the window while SMs are idle
+        span = (batch.block_table.shape[1] if m.window is None else (m.window + 2 * PAGE - 2) // PAGE
+                + (m.keep_first + PAGE - 1) // PAGE)
+        splits = max(1, min(span, 2 * 148 // (batch.T * m.kv_heads)))
+        part = None if splits == 1 else torch.empty(batch.T * m.heads * splits, 130, dtype=torch.float32, device=q.device)
+        ml = None if part is None else part.view(-1)[batch.T * m.heads * splits * 128:]
+        _lib.check_rc(L.b200_attn_decode_window(
+            _p(q), _p(k_cache), _p(v_cache), _p(batch.block_table), _p(batch.start), _p(out), _i(out.stride(0)), _p(part),
+            _p(ml), _i(batch.T), _i(m.heads), _i(m.kv_heads), _i(m.dim), _i(m.vdim), _i(m.k_ld), _i(m.v_ld),
+            _i(k_cache.shape[0] // PAGE), _i(batch.block_table.stride(0)), _i(splits), _i(window), _i(m.keep_first),
+            _i(int(m.sink)), _f(m.scale), _p(_lib.status_word(q.device)), _lib.stream_ptr()), "attn_decode_window")
+        return
+    if impl == "tiles":
+        assert fits, "sizes outside the tensor-core kernel"
+        ts, tq0, nt = batch.query_tiles(128 // rep)
+        _lib.check_rc(L.b200_attn_window(
+            _p(q), _p(k_cache), _p(v_cache), _p(batch.cu), _p(batch.start), _p(batch.block_table), _p(ts), _p(tq0), _i(nt),
+            _i(batch.T), _i(batch.block_table.stride(0)), _i(k_cache.shape[0] // PAGE), _p(out), _i(out.stride(0)),
+            _i(m.heads), _i(m.kv_heads), _i(m.dim), _i(m.vdim), _i(m.k_ld), _i(m.v_ld), _i(window), _i(m.keep_first),
+            _i(int(m.sink)), _f(m.scale), _p(_lib.status_word(q.device)), _lib.stream_ptr()), "attn_window")
+        return
     _lib.check_rc(L.b200_attn_ragged(
         _p(q), _p(k_cache), _p(v_cache), _p(batch.cu), _p(batch.start), _p(batch.tok_seq), _p(batch.block_table),
-        _i(batch.n), _i(T), _i(batch.block_table.stride(0)), _i(PAGE), _p(out), _i(out.stride(0)), _i(m.heads),
+        _i(batch.n), _i(batch.T), _i(batch.block_table.stride(0)), _i(PAGE), _p(out), _i(out.stride(0)), _i(m.heads),
         _i(m.kv_heads), _i(m.dim), _i(m.vdim), _i(m.k_ld), _i(m.v_ld), _i(window), _i(m.keep_first), _i(int(m.sink)),
-        _f(m.scale), f32, st()), "attn_ragged")
+        _f(m.scale), _f32(q.dtype), _lib.stream_ptr()), "attn_ragged")

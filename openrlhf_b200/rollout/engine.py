@@ -369,7 +369,8 @@ class RolloutEngine:
         for p in parts:
             out.append(flat[o:o + p.numel()])
             o += (p.numel() + 3) // 4 * 4
-        return StepBatch(out[0].long(), out[1], out[2], out[3], out[4], out[5], out[6], out[7].view(n, -1), n, T, max(lens))
+        return StepBatch(out[0].long(), out[1], out[2], out[3], out[4], out[5], out[6], out[7].view(n, -1), n, T, max(lens),
+                         lens=lens)
 
     @torch.no_grad()
     def _forward_tokens(self, items: list, mms: list | None = None):

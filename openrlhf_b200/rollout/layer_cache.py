@@ -51,4 +51,5 @@ class LayerCache:
     def copy_row(self, src: int, dst: list):
         for k, t in self._t.items():
             if self._place[k][4] == "row":
-                t[dst] = t[src]
+                for d in dst:
+                    t[d].copy_(t[src])
