@@ -81,6 +81,9 @@ def parse():
     ap.add_argument("--rollout-tp", type=int, default=None, help="tensor-parallel size of the rollout engines")
     ap.add_argument("--extras", default="auto", choices=["auto", "none"],
                     help="auto: after the default config, measure the other configs in child processes if time allows")
+    ap.add_argument("--serving", default=None, metavar="SIZES",
+                    help="instead: prefill and decode throughput of the hybrid design beside the dense transformer of equal "
+                         "size, e.g. 1b or 1b,8b (bench/serving.py); one GPU")
     return ap.parse_args()
 
 
@@ -192,6 +195,8 @@ def main():
     args = parse()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.serving:
+        return serving(args)
     import torch
     import torch.distributed as dist
 
@@ -361,6 +366,20 @@ def main():
         dist.destroy_process_group()
     if out is not None:
         print(json.dumps(out))
+    return 0
+
+
+def serving(args) -> int:
+    import torch
+
+    from bench.serving import run
+
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    res = run(args.serving.split(","), max(3, args.warmup), max(5, args.steps))
+    print(json.dumps({"metric": "serving throughput, prefill and decode tokens/s", "n_gpus": 1, "dtype": "bf16",
+                      "data": "synthetic token ids, random-init weights", "warmup": max(3, args.warmup),
+                      "steps": max(5, args.steps), "sizes": res, "clocks": sampler.stop()}))
     return 0
 
 

@@ -206,26 +206,28 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
       // ---- step sizes and the running sum of log2 decays
       const float dtv = dt_next;
       dt_next = tok + SC_Q < len ? dt[tok + SC_Q] : 0.f;
-      float cum = a2 * dtv;
+      // sums inside the row's block of 32 tokens, from its start up to t and behind t to its end (scanned both ways: a
+      // difference of prefix sums would lose the small distances behind a stretch of fast decay)
+      float pre = a2 * dtv, suf = pre;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
-        const float u = __shfl_up_sync(0xffffffffu, cum, o);
-        if (lane >= o) cum += u;
+        const float u = __shfl_up_sync(0xffffffffu, pre, o), v = __shfl_down_sync(0xffffffffu, suf, o);
+        if (lane >= o) pre += u;
+        if (lane + o < 32) suf += v;
       }
-      if (half == 0 && lane == 31) wtot[quarter] = cum;
+      suf = __shfl_down_sync(0xffffffffu, suf, 1);
+      if (lane == 31) suf = 0.f;
+      if (half == 0 && lane == 31) wtot[quarter] = pre;
       asm volatile("bar.sync 1, 256;" ::: "memory");
-      float total = 0.f, ref[4];                            // ref[q]: the sum at the end of the q-th 32 tokens
-#pragma unroll
-      for (int q = 0; q < 4; ++q) {
-        const float w = wtot[q];
-        if (q < quarter) cum += w;
-        total += w;
-        ref[q] = total;
-      }
-      // a block of 32 tokens in front of this row's weighs its token s with e^{ref - cum_s} dt_s, the same for all rows,
-      // and the row adds e^{cum_t - ref}; both exponents are <= 0
-      if (half == 0) wsm[t] = ex2((quarter == 0 ? ref[0] : quarter == 1 ? ref[1] : quarter == 2 ? ref[2] : ref[3]) - cum) * dtv;
-      const float w_own = cum - lg2(dtv);                   // for the diagonal block; dt = 0: +inf, the weight vanishes
+      const float b0 = wtot[0], b1 = wtot[1], b2 = wtot[2], b3 = wtot[3];
+      // from the end of block q (0, 1, 2) to this row's block, and from there to the end of the chunk
+      const float gap2 = 0.f, gap1 = quarter > 2 ? b2 : 0.f, gap0 = quarter > 2 ? b1 + b2 : quarter > 1 ? b1 : 0.f;
+      const float ahead = quarter == 0 ? b1 + b2 + b3 : quarter == 1 ? b2 + b3 : quarter == 2 ? b3 : 0.f;
+      const float cum = pre + (quarter == 0 ? 0.f : b0 + gap0), total = b0 + b1 + b2 + b3;
+      // a block of 32 tokens in front of this row's weighs its token s with e^{sum behind s} dt_s, the same for all rows,
+      // and the row adds the decay from the block's end to itself
+      if (half == 0) wsm[t] = ex2(suf) * dtv;
+      const float w_own = pre - lg2(dtv);                   // for the diagonal block; dt = 0: +inf, the weight vanishes
       // ---- S: bf16 hi / lo rows for the read-out, decayed in place for the update
       tmem_ld_32x32b_x32(tm_s + lane_addr + c0, r);
       tmem_ld_wait();
@@ -265,7 +267,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
           const int q = half + 2 * u;
           if (q < quarter) {
             tmem_ld_32x32b_x32(tm_g + lane_addr + q * 32, r);
-            const float rs = ex2(cum - (q == 0 ? ref[0] : q == 1 ? ref[1] : ref[2]));
+            const float rs = ex2(pre + (q == 0 ? gap0 : q == 1 ? gap1 : gap2));
             tmem_ld_wait();
 #pragma unroll
             for (int j = 0; j < 32; j += 4) {
@@ -279,8 +281,8 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
 #pragma unroll
             for (int j = 0; j < 32; j += 2) {
               const float w0 = __shfl_sync(0xffffffffu, w_own, j), w1 = __shfl_sync(0xffffffffu, w_own, j + 1);
-              const float a = j <= lane ? ex2(cum - w0) * __uint_as_float(r[j]) : 0.f;
-              const float b = j + 1 <= lane ? ex2(cum - w1) * __uint_as_float(r[j + 1]) : 0.f;
+              const float a = j <= lane ? ex2(pre - w0) * __uint_as_float(r[j]) : 0.f;
+              const float b = j + 1 <= lane ? ex2(pre - w1) * __uint_as_float(r[j + 1]) : 0.f;
               split2(a, b, m_hi[u][j / 2], m_lo[u][j / 2]);
             }
           } else {
@@ -312,7 +314,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
       // ---- weighted inputs into the S tiles (their MMAs are complete); x stays in registers for the skip term
       uint4 x[4];
       {
-        const float w = ex2(total - cum) * dtv;
+        const float w = ex2(suf + ahead) * dtv;
         ok = ok && mbar_wait(x_full, ph, p.status, ERR_TIMEOUT_FULL);
         const uint8_t* xs = smem + ScSmem::X_OFF;
         uint8_t* w_hi = smem + ScSmem::S_OFF;

@@ -79,8 +79,9 @@ def feed(eng, toks, cuts, key="s"):
     return torch.cat(out)
 
 
-def rel_rms(got, want):
-    """Root mean square over the vocabulary of the difference (mean taken off), over the logits' own spread: worst row."""
+def rel_rms(got, want, quantile=1.0):
+    """Root mean square over the vocabulary of the difference (mean taken off), over the logits' own spread: worst row, or
+    a quantile of the rows. (In bf16 a few positions of a random model amplify rounding, wherever its kernels run.)"""
     d = got.double() - want.double()
     d = d - d.mean(-1, keepdim=True)
-    return float((d.pow(2).mean(-1).sqrt() / want.double().std()).max())
+    return float((d.pow(2).mean(-1).sqrt() / want.double().std()).quantile(quantile))
