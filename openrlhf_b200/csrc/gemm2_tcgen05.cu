@@ -50,6 +50,9 @@ struct Gemm2Params {
   int swiglu, sw_half;
   __nv_bfloat16* C2;
   int ldc2;
+  // Split output with an activation (bf16 outputs): columns from act_col0 on (a multiple of 32, > 0) leave as relu(x)^2
+  // in C2[M, ldc2], the columns before it as they are in C[M, ldc]
+  int act_col0;
   // LM-head backward recomputation: C receives d logits = g / T * (onehot(label) - exp(z / T - lse)) as bf16
   // (z = the product, one row per token); see GemmParams::lp_mode in gemm_tcgen05.cu.
   int lp_mode;
@@ -355,7 +358,11 @@ gemm2_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_consta
               }
             }
           } else {
-            __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)row * p.ldc + col0;
+            // a 32-column chunk lies on one side of act_col0
+            const bool act = p.act_col0 > 0 && col0 >= p.act_col0;
+            const bool wide = act ? wide_c2 : wide_c;
+            __nv_bfloat16* crow = act ? p.C2 + (size_t)row * p.ldc2 + (col0 - p.act_col0)
+                                      : reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)row * p.ldc + col0;
 #pragma unroll
             for (int j = 0; j < 32; j += 16) {
               uint4 o[2];
@@ -395,13 +402,17 @@ gemm2_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_consta
                       v[2 * q + 1] += f.y;
                     }
                   }
+                  if (act) {
+#pragma unroll
+                    for (int q = 0; q < 8; ++q) { const float u = fmaxf(v[q], 0.f); v[q] = u * u; }
+                  }
                   o[hh].x = pack_bf16x2(v[0], v[1]);
                   o[hh].y = pack_bf16x2(v[2], v[3]);
                   o[hh].z = pack_bf16x2(v[4], v[5]);
                   o[hh].w = pack_bf16x2(v[6], v[7]);
                 }
               }
-              if (wide_c && col0 + j + 16 <= p.N) {
+              if (wide && col0 + j + 16 <= p.N) {
                 st_global_256(crow + j, o[0], o[1]);
               } else {
                 if (col0 + j < p.N) *reinterpret_cast<uint4*>(crow + j) = o[0];
@@ -457,9 +468,10 @@ static int g2_sm_count = 0;
 
 // Same contract as b200_gemm_bf16 (bf16 operands, bf16 or fp32 output) without split-K slabs, on CTA pairs.
 // bn: 128 or 256 (0: 256).
-extern "C" int b200_gemm2_bf16(const void* A, const void* B, void* C, const void* bias, const void* residual, int M,
-                               int N, int K, int lda, int ldb, int ldc, int a_mn, int b_mn, int out_f32, int accumulate,
-                               int k_splits, float alpha, int bn, int* status, void* stream_) {
+static int gemm2_bf16_impl(const void* A, const void* B, void* C, const void* bias, const void* residual, int M,
+                           int N, int K, int lda, int ldb, int ldc, int a_mn, int b_mn, int out_f32, int accumulate,
+                           int k_splits, float alpha, int bn, int act_col0, void* C2, int ldc2, int* status,
+                           void* stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((lda % 8) || (ldb % 8) || (ldc % (out_f32 ? 4 : 8)) || (N % (out_f32 ? 4 : 8))) return -10;
@@ -486,6 +498,7 @@ extern "C" int b200_gemm2_bf16(const void* A, const void* B, void* C, const void
   p.residual = reinterpret_cast<const __nv_bfloat16*>(residual);
   p.M = M; p.N = N; p.K = K; p.ldc = ldc; p.out_f32 = out_f32; p.accumulate = accumulate; p.k_splits = k_splits;
   p.alpha = alpha; p.status = status;
+  p.act_col0 = act_col0; p.C2 = reinterpret_cast<__nv_bfloat16*>(C2); p.ldc2 = ldc2;
 #define B200_DISPATCH2(BN_)                                                                \
   if (!a_mn && !b_mn) return launch2<BN_, false, false>(ta, tb, p, g2_sm_count, stream);   \
   if (!a_mn && b_mn) return launch2<BN_, false, true>(ta, tb, p, g2_sm_count, stream);     \
@@ -494,6 +507,21 @@ extern "C" int b200_gemm2_bf16(const void* A, const void* B, void* C, const void
   if (bn == 256) { B200_DISPATCH2(256) }
   B200_DISPATCH2(128)
 #undef B200_DISPATCH2
+}
+
+extern "C" int b200_gemm2_bf16(const void* A, const void* B, void* C, const void* bias, const void* residual, int M,
+                               int N, int K, int lda, int ldb, int ldc, int a_mn, int b_mn, int out_f32, int accumulate,
+                               int k_splits, float alpha, int bn, int* status, void* stream_) {
+  return gemm2_bf16_impl(A, B, C, bias, residual, M, N, K, lda, ldb, ldc, a_mn, b_mn, out_f32, accumulate, k_splits, alpha,
+                         bn, 0, nullptr, 0, status, stream_);
+}
+
+// Split output with relu^2 on the columns from act_col0 on; same contract as b200_gemm_bf16_relu2.
+extern "C" int b200_gemm2_bf16_relu2(const void* A, const void* B, void* C, void* C2, int M, int N, int K, int lda, int ldb,
+                                     int ldc, int ldc2, int act_col0, int bn, int* status, void* stream_) {
+  if (act_col0 <= 0 || act_col0 % 32 || N % 32 || ldc2 % 8 || (reinterpret_cast<uintptr_t>(C2) & 15)) return -10;
+  return gemm2_bf16_impl(A, B, C, nullptr, nullptr, M, N, K, lda, ldb, ldc, 0, 0, 0, 0, 1, 1.f, bn, act_col0, C2, ldc2,
+                         status, stream_);
 }
 
 

@@ -57,6 +57,9 @@ struct GemmParams {
   int sw_half;
   __nv_bfloat16* C2;
   int ldc2;
+  // Split output with an activation (bf16 outputs): columns from act_col0 on (a multiple of 32, > 0) leave as relu(x)^2
+  // in C2[M, ldc2], the columns before it as they are in C[M, ldc]
+  int act_col0;
   // LM-head epilogues (K-LMHEAD): the product is logits[tokens, vocabulary], never written as such.
   //   lp_mode 1 (forward): every tile reduces its BN columns to per-row softmax partials
   //       lp_partial[(n_blk * M + row) * 8 + {0: max z, 1: sum exp((z - max) / T), 2: sum exp(z - max),
@@ -465,7 +468,11 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
               }
             }
           } else {
-            __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)row * p.ldc + col0;
+            // a 32-column chunk lies on one side of act_col0
+            const bool act = p.act_col0 > 0 && col0 >= p.act_col0;
+            const bool wide = act ? wide_c2 : wide_c;
+            __nv_bfloat16* crow = act ? p.C2 + (size_t)row * p.ldc2 + (col0 - p.act_col0)
+                                      : reinterpret_cast<__nv_bfloat16*>(p.C) + (size_t)row * p.ldc + col0;
 #pragma unroll
             for (int j = 0; j < 32; j += 16) {
               uint4 o[2];
@@ -506,13 +513,17 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constan
                       v[2 * q + 1] += f.y;
                     }
                   }
+                  if (act) {
+#pragma unroll
+                    for (int q = 0; q < 8; ++q) { const float u = fmaxf(v[q], 0.f); v[q] = u * u; }
+                  }
                   o[hh].x = pack_bf16x2(v[0], v[1]);
                   o[hh].y = pack_bf16x2(v[2], v[3]);
                   o[hh].z = pack_bf16x2(v[4], v[5]);
                   o[hh].w = pack_bf16x2(v[6], v[7]);
                 }
               }
-              if (wide_c && col0 + j + 16 <= p.N) {
+              if (wide && col0 + j + 16 <= p.N) {
                 st_global_256(crow + j, o[0], o[1]);          // one full 32-byte sector per thread
               } else {
                 if (col0 + j < p.N) *reinterpret_cast<uint4*>(crow + j) = o[0];
@@ -676,10 +687,10 @@ extern "C" int b200_set_pdl(int on) { return b200::g_pdl_mode.exchange(on ? 1 : 
 
 // C-callable entry point. a_mn / b_mn select the operand layouts documented at the top of this file.
 // lda / ldb are the row strides (elements) of the tensors as they sit in memory. Returns 0 on a successful launch.
-extern "C" int b200_gemm_bf16(const void* A, const void* B, void* C, const void* bias, const void* residual, int M,
-                              int N, int K, int lda, int ldb, int ldc, int a_mn, int b_mn, int out_f32,
-                              int accumulate, int k_splits, long long split_stride, float alpha, int bn, int* status,
-                              void* stream_) {
+static int gemm_bf16_impl(const void* A, const void* B, void* C, const void* bias, const void* residual, int M,
+                          int N, int K, int lda, int ldb, int ldc, int a_mn, int b_mn, int out_f32,
+                          int accumulate, int k_splits, long long split_stride, float alpha, int bn, int act_col0,
+                          void* C2, int ldc2, int* status, void* stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if ((lda % 8) || (ldb % 8) || (ldc % (out_f32 ? 4 : 8)) || (N % (out_f32 ? 4 : 8))) return -10;
@@ -709,6 +720,7 @@ extern "C" int b200_gemm_bf16(const void* A, const void* B, void* C, const void*
   p.out_f32 = out_f32; p.accumulate = accumulate; p.k_splits = k_splits; p.split_stride = split_stride; p.alpha = alpha; p.status = status;
   p.n_peer_c = 0; p.ag_world = 0; p.ag_rows = 0;
   p.b_static = pdl_static_weights() ? 1 : 0;
+  p.act_col0 = act_col0; p.C2 = reinterpret_cast<__nv_bfloat16*>(C2); p.ldc2 = ldc2;
   for (int i = 0; i < 8; ++i) p.peer_c[i] = nullptr;
   static PeerMaps no_peers;
 #define B200_DISPATCH(BN_)                                                                            \
@@ -720,6 +732,23 @@ extern "C" int b200_gemm_bf16(const void* A, const void* B, void* C, const void*
   if (bn == 128) { B200_DISPATCH(128) }
   B200_DISPATCH(64)
 #undef B200_DISPATCH
+}
+
+extern "C" int b200_gemm_bf16(const void* A, const void* B, void* C, const void* bias, const void* residual, int M,
+                              int N, int K, int lda, int ldb, int ldc, int a_mn, int b_mn, int out_f32,
+                              int accumulate, int k_splits, long long split_stride, float alpha, int bn, int* status,
+                              void* stream_) {
+  return gemm_bf16_impl(A, B, C, bias, residual, M, N, K, lda, ldb, ldc, a_mn, b_mn, out_f32, accumulate, k_splits,
+                        split_stride, alpha, bn, 0, nullptr, 0, status, stream_);
+}
+
+// A [M, K], B [N, K] bf16: C[M, act_col0] receives the first act_col0 columns of A B^T, C2[M, N - act_col0] relu^2 of the
+// rest. act_col0 and N are multiples of 32.
+extern "C" int b200_gemm_bf16_relu2(const void* A, const void* B, void* C, void* C2, int M, int N, int K, int lda, int ldb,
+                                    int ldc, int ldc2, int act_col0, int bn, int* status, void* stream_) {
+  if (act_col0 <= 0 || act_col0 % 32 || N % 32 || ldc2 % 8 || (reinterpret_cast<uintptr_t>(C2) & 15)) return -10;
+  return gemm_bf16_impl(A, B, C, nullptr, nullptr, M, N, K, lda, ldb, ldc, 0, 0, 0, 0, 1, 0, 1.f, bn, act_col0, C2, ldc2,
+                        status, stream_);
 }
 
 

@@ -70,6 +70,40 @@ rmsnorm_f32_kernel(float* __restrict__ x, const float* __restrict__ ws, int spli
   }
 }
 
+// Long batches without slabs: one warp per row, the row in registers (ld up to 32 * 4 * NV).
+template <typename T, int NV>
+__global__ void __launch_bounds__(HY_THREADS)
+rmsnorm_f32_warp_kernel(const float* __restrict__ x, const T* __restrict__ w, T* __restrict__ y, int M, int n, int ld,
+                        float eps) {
+  const int lane = threadIdx.x & 31;
+  for (int m = blockIdx.x * (HY_THREADS / 32) + (threadIdx.x >> 5); m < M; m += gridDim.x * (HY_THREADS / 32)) {
+    float f[NV][4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 32 + lane) * 4;
+      if (c < ld) load4(x + (size_t)m * ld + c, f[i]);
+      else f[i][0] = f[i][1] = f[i][2] = f[i][3] = 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+#pragma unroll
+      for (int k = 0; k < 4; ++k) ss += f[i][k] * f[i][k];
+    const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)n + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 32 + lane) * 4;
+      if (c < ld) {
+        float g[4];
+        load4(w + c, g);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) f[i][k] = f[i][k] * rstd * g[k];
+        store4(y + (size_t)m * ld + c, f[i]);
+      }
+    }
+  }
+}
+
 // ------------------------------------------------------------------ logits <- cap * tanh(logits / cap)
 __global__ void softcap_kernel(float* __restrict__ x, long long n4, float cap, float inv_cap) {
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < n4; i += (long long)gridDim.x * blockDim.x) {
@@ -86,6 +120,64 @@ __global__ void softcap_kernel(float* __restrict__ x, long long n4, float cap, f
 // layer's cache. Channels [0, rot) of a head rotate in pairs (i, i + rot/2) with the (cos, sin) row of the token's
 // position; the rest pass. q -> q_out [T, H, dk_ld]; k, v -> cache slot. Cache and q rows are padded to dk_ld / dv_ld
 // (their padding stays zero). One thread per element pair; ff columns are squared-ReLU'd into `ff_dst`.
+// The same, four channels at a time (rot / 2, dk - rot and dv multiples of 4).
+template <typename T>
+__global__ void __launch_bounds__(HY_THREADS)
+rope_write4_kernel(const Proj<T> src, const int* __restrict__ pos, const int* __restrict__ slots,
+                   const float2* __restrict__ table, int max_pos, T* __restrict__ q_out, T* __restrict__ k_cache,
+                   T* __restrict__ v_cache, int n_tok, int H, int G, int dk, int dv, int dk_ld, int dv_ld, int rot,
+                   int ff_col, int ff, T* __restrict__ ff_dst, int ff_ld) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int half = rot >> 1;
+  const int per_qk = (half + (dk - rot)) >> 2;
+  const int n_qk = (H + G) * per_qk, n_v = (G * dv) >> 2, n_f = ff >> 2;
+  const int per_tok = n_qk + n_v + n_f;
+  const int step = gridDim.x * HY_THREADS;
+  const long long total = (long long)n_tok * per_tok;
+  for (long long idx = blockIdx.x * (long long)HY_THREADS + threadIdx.x; idx < total; idx += step) {
+    const int t = (int)(idx / per_tok);
+    int e = (int)(idx - (long long)t * per_tok);
+    float u[4];
+    if (e < n_qk) {
+      const int head = e / per_qk, i = (e - head * per_qk) * 4;
+      T* dst = head < H ? q_out + ((size_t)t * H + head) * dk_ld : k_cache + ((size_t)slots[t] * G + (head - H)) * dk_ld;
+      const int c0 = head * dk;
+      if (i < half) {
+        float v[4], a[4], b[4], cs[8];
+        src.get4(t, c0 + i, u);
+        src.get4(t, c0 + i + half, v);
+        int p = pos[t];
+        p = p < 0 ? 0 : (p >= max_pos ? max_pos - 1 : p);
+        const float* row = reinterpret_cast<const float*>(table + (size_t)p * half + i);
+        load4(row, cs);
+        load4(row + 4, cs + 4);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          a[k] = u[k] * cs[2 * k] - v[k] * cs[2 * k + 1];
+          b[k] = v[k] * cs[2 * k] + u[k] * cs[2 * k + 1];
+        }
+        store4(dst + i, a);
+        store4(dst + i + half, b);
+      } else {
+        src.get4(t, c0 + i + half, u);
+        store4(dst + i + half, u);
+      }
+    } else if (e < n_qk + n_v) {
+      e = (e - n_qk) * 4;
+      const int g = e / dv;
+      src.get4(t, (H + G) * dk + e, u);
+      store4(v_cache + ((size_t)slots[t] * G + g) * dv_ld + (e - g * dv), u);
+    } else {
+      e = (e - n_qk - n_v) * 4;
+      src.get4(t, ff_col + e, u);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) { const float r = fmaxf(u[k], 0.f); u[k] = r * r; }
+      store4(ff_dst + (size_t)t * ff_ld + e, u);
+    }
+  }
+}
+
 template <typename T>
 __global__ void rope_write_kernel(const Proj<T> src, const int* __restrict__ pos, const int* __restrict__ slots,
                                   const float2* __restrict__ table, int max_pos, T* __restrict__ q_out,
@@ -224,6 +316,13 @@ extern "C" int b200_rmsnorm_f32(float* x, const float* ws, int splits, long long
   const int grid = M < 148 * 8 ? M : 148 * 8;
   const size_t smem = (size_t)ld * sizeof(float);
   cudaError_t e;
+  if (!f32 && ws == nullptr && rows == nullptr && M >= 1024 && ld <= 4096) {
+    typedef __nv_bfloat16 B16;
+    const int blocks = (M + 7) / 8 < 148 * 8 ? (M + 7) / 8 : 148 * 8;
+    if (ld <= 2048) rmsnorm_f32_warp_kernel<B16, 16><<<blocks, HY_THREADS, 0, HY_STREAM(stream)>>>(x, (const B16*)w, (B16*)y, M, n, ld, eps);
+    else rmsnorm_f32_warp_kernel<B16, 32><<<blocks, HY_THREADS, 0, HY_STREAM(stream)>>>(x, (const B16*)w, (B16*)y, M, n, ld, eps);
+    return HY_OK();
+  }
   if (f32) e = launch_pdl(rmsnorm_f32_kernel<float>, dim3(grid), dim3(HY_THREADS), smem, HY_STREAM(stream), x, ws, splits,
                           slab, rows, (const float*)w, (float*)y, M, n, ld, eps);
   else e = launch_pdl(rmsnorm_f32_kernel<__nv_bfloat16>, dim3(grid), dim3(HY_THREADS), smem, HY_STREAM(stream), x, ws,
@@ -245,12 +344,16 @@ extern "C" int b200_rope_write(const void* p, const float* ws, int splits, long 
   if (n_tok <= 0) return 0;
   if (rot % 2 || rot > dk || dk_ld < dk || dv_ld < dv || ff % 4 || ff_col % 4 || ld % 4 || ff_ld % 4 || slab % 4) return -10;
   const long long work = (long long)n_tok * ((H + G) * (rot / 2 + dk - rot) + G * dv + ff / 4);
-  const int grid = hy_grid(work, 148 * 16);
+  const bool vec = rot % 8 == 0 && (dk - rot) % 4 == 0 && dv % 4 == 0;
+  const int grid = hy_grid(vec ? work / 4 : work, 148 * 16);
   cudaError_t e;
 #define ROPE_ARGS(TT)                                                                                                 \
   make_proj<TT>(p, ws, splits, slab, ld), pos, slots, (const float2*)table, max_pos, (TT*)q_out, (TT*)k_cache,        \
       (TT*)v_cache, n_tok, H, G, dk, dv, dk_ld, dv_ld, rot, ff_col, ff, (TT*)ff_dst, ff_ld
-  if (f32) e = launch_pdl(rope_write_kernel<float>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(float));
+  if (vec) {
+    if (f32) e = launch_pdl(rope_write4_kernel<float>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(float));
+    else e = launch_pdl(rope_write4_kernel<__nv_bfloat16>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(__nv_bfloat16));
+  } else if (f32) e = launch_pdl(rope_write_kernel<float>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(float));
   else e = launch_pdl(rope_write_kernel<__nv_bfloat16>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(__nv_bfloat16));
 #undef ROPE_ARGS
   return e == cudaSuccess ? 0 : -3;

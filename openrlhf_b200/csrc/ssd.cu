@@ -75,6 +75,67 @@ conv_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, const
   }
 }
 
+// The same for long batches: a thread slides down a run of tokens with the last TAPS - 1 inputs of its four channels in
+// registers, so every input is read once (and TAPS - 1 once more per run). A run may cross into another sequence.
+constexpr int CONV_RUN = 32, CONV_BATCH = 8;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256)
+conv_run_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, const T* __restrict__ w,
+                const T* __restrict__ bias, T* __restrict__ out, const SsdDims d) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= d.cc) return;
+  const int t0 = blockIdx.y * CONV_RUN, t1 = min(b.T, t0 + CONV_RUN);
+  float wt[TAPS][4], bs[4], hist[TAPS][4];
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    bs[q] = to_f(bias[c + q]);
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k) wt[k][q] = to_f(w[(size_t)(c + q) * TAPS + k]);
+  }
+  int seq = -1;
+  for (int t = t0; t < t1; t += CONV_BATCH) {
+    float u[CONV_BATCH][4];
+#pragma unroll
+    for (int j = 0; j < CONV_BATCH; ++j)
+      if (t + j < t1) load4(src.p + (size_t)(t + j) * src.ld + d.inner + c, u[j]);
+#pragma unroll
+    for (int j = 0; j < CONV_BATCH; ++j) {
+      if (t + j >= t1) break;
+      const int i = b.tok_seq[t + j];
+      if (i != seq) {                                     // the run's first token, or another sequence begins
+        seq = i;
+        const int row0 = b.cu[i], o = t + j - row0;
+#pragma unroll
+        for (int k = 1; k < TAPS; ++k)
+          conv_input<T, 4>(src, ring + (size_t)b.row[i] * d.taps * d.cc, row0, o - (TAPS - k), b.start[i], TAPS, d.cc,
+                           d.inner, c, hist[k]);          // hist[k]: the input TAPS - k tokens back
+      }
+      float acc[4];
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        acc[q] = bs[q];
+#pragma unroll
+        for (int k = 1; k < TAPS; ++k) acc[q] = fmaf(wt[k - 1][q], hist[k][q], acc[q]);
+        acc[q] = silu_f(fmaf(wt[TAPS - 1][q], u[j][q], acc[q]));
+#pragma unroll
+        for (int k = 1; k + 1 < TAPS; ++k) hist[k][q] = hist[k + 1][q];
+        if (TAPS > 1) hist[TAPS - 1][q] = u[j][q];
+      }
+      store4(out + (size_t)(t + j) * d.cc + c, acc);
+    }
+  }
+}
+
+// dt[h, t] = softplus(proj + dt_bias[h]) for the run kernel: 32 tokens per block, written in whole lines.
+template <typename T>
+__global__ void __launch_bounds__(256)
+dt_kernel(const Proj<T> src, const T* __restrict__ dt_bias, float* __restrict__ dt, int n_tok, const SsdDims d) {
+  const int t = blockIdx.x * 32 + (threadIdx.x & 31);
+  if (t >= n_tok) return;
+  for (int h = threadIdx.x >> 5; h < d.H; h += 8)
+    dt[(size_t)h * n_tok + t] = softplus_f(src.get_raw(t, d.inner + d.cc + h) + to_f(dt_bias[h]));
+}
+
 // The last taps - 1 inputs of every portion go to the ring (after conv_kernel has read the old entries).
 template <typename T>
 __global__ void conv_ring_kernel(const Proj<T> src, const Ragged b, T* __restrict__ ring, const SsdDims d) {
@@ -230,6 +291,18 @@ template <typename T>
 static int launch_conv(const Proj<T>& src, const Ragged& b, T* ring, const T* w, const T* bias, const T* dt_bias, T* out,
                        float* dt, const SsdDims& d, cudaStream_t st) {
   const bool vec = d.cc % 4 == 0 && d.inner % 4 == 0 && src.ld % 4 == 0 && src.slab % 4 == 0;
+  if (vec && src.ws == nullptr && b.T >= 64 && d.taps >= 1 && d.taps <= 4) {
+    const dim3 grid((d.cc / 4 + 255) / 256, (b.T + CONV_RUN - 1) / CONV_RUN);
+    if (grid.y > 65535) return -10;
+    if (d.taps == 1) conv_run_kernel<T, 1><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
+    else if (d.taps == 2) conv_run_kernel<T, 2><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
+    else if (d.taps == 3) conv_run_kernel<T, 3><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
+    else conv_run_kernel<T, 4><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
+    dt_kernel<T><<<(b.T + 31) / 32, 256, 0, st>>>(src, dt_bias, dt, b.T, d);
+    if (cudaGetLastError() != cudaSuccess) return -3;
+    if (d.taps > 1) conv_ring_kernel<T><<<dim3((d.cc + 255) / 256, b.n), 256, 0, st>>>(src, b, ring, d);
+    return cudaGetLastError() == cudaSuccess ? 0 : -3;
+  }
   const long long work = (long long)b.T * ((vec ? d.cc / 4 : d.cc) + d.H);
   long long blocks = (work + 255) / 256;
   if (blocks > 148 * 32) blocks = 148 * 32;

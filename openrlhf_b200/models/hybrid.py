@@ -133,16 +133,17 @@ class HybridLM(FlatModel):
         for i, layer in enumerate(cfg.layers):
             m = layer.mixer
             pre = f"layers.{i}."
-            p = H.project(h, self.p(pre + "w1.weight"))
             new = torch.empty if m.out_cols == layer.out_pad else torch.zeros
             a = new(batch.T, layer.out_pad + layer.ff_pad, dtype=h.dtype, device=h.device)
+            p = H.project(h, self.p(pre + "w1.weight"), layer.in_pad, a[:, layer.out_pad:])
+            ff = p.cols - layer.in_pad            # 0: the projection has already turned the feed-forward columns
             if isinstance(m, Mamba2Spec):
                 H.mamba2(p, m, self._mamba[i], cache.get(i, "ring"), cache.get(i, "state"), batch, eps, a, layer.out_pad,
-                         layer.in_pad, layer.ff_pad)
+                         layer.in_pad, ff)
             else:
                 src = i if m.kv_from is None else m.kv_from
                 H.window_attention(p, m, self._table(m), cache.get(src, "k"), cache.get(src, "v"), batch, a, layer.out_pad,
-                                   layer.in_pad, layer.ff_pad)
+                                   layer.in_pad, ff)
             # the norm that follows rides on the residual add (the last layer's too, when every row's logits are wanted)
             nxt = self.p(f"layers.{i + 1}.norm1.weight") if i < last else (self.p("norm.weight") if want is None else None)
             h = H.add_norm(x, a, self.p(pre + "w2.weight"), nxt, n, eps)

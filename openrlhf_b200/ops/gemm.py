@@ -126,6 +126,22 @@ def gemm_swiglu(x: torch.Tensor, w: torch.Tensor, want_gate_up: bool = False, bn
     return y, gu
 
 
+def gemm_relu2(x: torch.Tensor, w: torch.Tensor, col0: int, act_out: torch.Tensor) -> torch.Tensor:
+    """x [M, K] @ w [N, K]^T with the columns from `col0` on (a multiple of 32, like N) leaving the epilogue as relu(x)^2
+    into `act_out` [M, >= N - col0] (a view of wider rows is fine). Returns the first `col0` columns [M, col0]."""
+    assert x.dtype == w.dtype == act_out.dtype == torch.bfloat16 and x.stride(1) == w.stride(1) == act_out.stride(1) == 1
+    M, K = x.shape
+    N = w.shape[0]
+    assert w.shape[1] == K and act_out.shape[0] == M and act_out.shape[1] >= N - col0
+    out = torch.empty(M, col0, dtype=torch.bfloat16, device=x.device)
+    fn = _lib.lib().b200_gemm2_bf16_relu2 if _use_pair_kernel(M, N, K, 1, 0, 0) else _lib.lib().b200_gemm_bf16_relu2
+    rc = fn(_lib.ptr(x), _lib.ptr(w), _lib.ptr(out), _lib.ptr(act_out), ctypes.c_int(M), ctypes.c_int(N), ctypes.c_int(K),
+            ctypes.c_int(x.stride(0)), ctypes.c_int(w.stride(0)), ctypes.c_int(col0), ctypes.c_int(act_out.stride(0)),
+            ctypes.c_int(col0), ctypes.c_int(0), _lib.ptr(_lib.status_word(x.device)), _lib.stream_ptr())
+    _lib.check_rc(rc, "gemm_relu2")
+    return out
+
+
 def swiglu_fusable(intermediate: int) -> bool:
     """The fused kernel pairs 128-row (or 64-row) blocks of the gate and up matrices."""
     return intermediate % 128 == 0

@@ -104,9 +104,10 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, n: int, eps: float, rows: torch.Te
 SMALL_M = 256      # up to this many tokens a projection is split along K into fp32 slabs
 
 
-def project(h: torch.Tensor, w: torch.Tensor) -> Projection:
-    """h [T, K] @ w[N, K]^T for consumers that take a ``Projection``."""
-    from .gemm import gemm, gemm_to_workspace
+def project(h: torch.Tensor, w: torch.Tensor, act_col: int = 0, act_out: torch.Tensor | None = None) -> Projection:
+    """h [T, K] @ w[N, K]^T for consumers that take a ``Projection``. With `act_out`, columns from `act_col` on may leave
+    as relu^2 into it; the returned projection then has only `act_col` columns, otherwise its consumer does it."""
+    from .gemm import gemm, gemm_relu2, gemm_to_workspace
 
     T, N = h.shape[0], w.shape[0]
     if not h.is_cuda:
@@ -116,6 +117,8 @@ def project(h: torch.Tensor, w: torch.Tensor) -> Projection:
     if T <= SMALL_M:
         ws, s = gemm_to_workspace(h, w)
         return Projection(None, ws, s, T, N, h.dtype)
+    if act_out is not None and N > act_col:
+        return Projection(gemm_relu2(h, w, act_col, act_out), None, 1, T, act_col, h.dtype)
     return Projection(gemm(h, w), None, 1, T, N, h.dtype)
 
 
