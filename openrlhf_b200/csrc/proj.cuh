@@ -106,7 +106,7 @@ inline Ragged make_ragged(const int* cu, const int* start, const int* row, const
   return r;
 }
 
-__device__ __forceinline__ float silu_f(float v) { return v / (1.f + __expf(-v)); }
+__device__ __forceinline__ float silu_f(float v) { return __fdividef(v, 1.f + __expf(-v)); }
 // log(1 + e^x) without overflow; both branches keep the relative accuracy of small results.
 __device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 

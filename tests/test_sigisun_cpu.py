@@ -217,3 +217,30 @@ def test_the_comparison_notices_a_wrong_mechanism(case, mistake, monkeypatch):
         f = O.group_rms_norm
         monkeypatch.setattr(O, "group_rms_norm", lambda x, wt, g, e: f(x, wt, g, e * 1000))
     assert rel_rms(O.forward(cfg, w, toks), right) > 2e-4
+
+
+def test_generate_command_line(tmp_path, capsys):
+    from openrlhf_b200.cli.generate import main
+
+    cfg = CONFIGS["ssm"]
+    w = write_checkpoint(tmp_path / "model", cfg, seed=6)
+    prompts = [tokens(cfg, 9, 1), tokens(cfg, 30, 2)]
+    (tmp_path / "in.jsonl").write_text(json.dumps(prompts[0]) + "\n" + json.dumps({"tokens": prompts[1]}) + "\n")
+    assert main(["--model", str(tmp_path / "model"), "--input", str(tmp_path / "in.jsonl"), "--device", "cpu", "--dtype",
+                 "float32", "--max_new_tokens", "5", "--n_samples", "2"]) == 0
+    rows = [json.loads(x) for x in capsys.readouterr().out.splitlines()]
+    assert [(r["prompt"], r["sample"]) for r in rows] == [(0, 0), (0, 1), (1, 0), (1, 1)]
+    for r in rows:
+        assert r["tokens"] == _greedy(cfg, w, prompts[r["prompt"]], 5) and r["finish_reason"] == "length"
+    assert main(["--model", "tiny-sigisun", "--input", str(tmp_path / "in.jsonl"), "--device", "cpu",
+                 "--max_new_tokens", "2"]) == 0
+
+
+def test_component_build_lists_existing_sources():
+    import os
+
+    from openrlhf_b200.csrc import build
+
+    for name in build.COMPONENTS:
+        assert all(os.path.exists(p) for p in build.sources(name))
+    assert build.PRECISE <= {os.path.basename(p) for p in build.sources()}
