@@ -74,7 +74,7 @@ def _time(fn, iters: int, flush: bool | None = None) -> float:
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--kernel", required=True, choices=["gemm", "gemm_fp8", "gemm_splitk", "gemm_swiglu", "decode_attn", "attn_fwd", "attn_bwd", "logprob", "logprob_bwd",
-                                                         "rmsnorm", "adamw", "decode_step", "decode_gemms", "sample", "ppo_loss", "gae"])
+                                                         "rmsnorm", "adamw", "decode_step", "decode_gemms", "sample", "ppo_loss", "gae", "hybrid"])
     ap.add_argument("--top-p", type=float, default=1.0, help="sample: nucleus threshold (1.0: plain Gumbel-max pass)")
     ap.add_argument("--model", default="qwen2.5-1.5b", help="decode_step: model preset")
     ap.add_argument("--layers", type=int, default=0, help="decode_step: cut the preset to this many layers (0: all)")
@@ -89,6 +89,7 @@ def main():
     ap.add_argument("--hkv", type=int, default=2)
     ap.add_argument("--splits", type=int, default=1)
     ap.add_argument("--bn", type=int, default=0, help="GEMM tile width (0: heuristic)")
+    ap.add_argument("--seqs", type=int, default=4, help="hybrid: sequences the --m prompt tokens are split into")
     ap.add_argument("--iters", type=int, default=10)
     ap.add_argument("--graph", type=int, default=0, help="time N back-to-back launches inside one CUDA graph")
     ap.add_argument("--no-flush", action="store_true", help="do not flush L2 between timed launches")
@@ -323,6 +324,9 @@ def main():
         print(f"decode_step {a.model} layers{cfg.num_hidden_layers} B{B} ctx{ctx}: {t * 1e3:.3f} ms per step over {n} "
               f"steps, {(wbytes + kvbytes) / t / 1e9:.0f} GB/s of weights + KV ({(wbytes + kvbytes) / t / 1e9 / hbm:.2f} "
               f"{tag} HBM), launches per graph {eng.graph_launches}, dependent-launch chain {a.pdl}")
+    elif a.kernel == "hybrid":
+        from bench.hybrid_kernels import run as hybrid_run
+        hybrid_run(a.model, a.m, a.seqs, a.batch, a.ctx, lambda fn: _time(fn, a.iters), hbm, tf, tag)
     elif a.kernel == "attn_fwd":
         T, Hq, Hkv, L = a.m, a.hq, a.hkv, a.ctx
         qkv = torch.randn(T, (Hq + 2 * Hkv) * 128, device=dev, dtype=torch.bfloat16)

@@ -32,7 +32,7 @@ NVCC_FLAGS = [
 PRECISE = {"hybrid_ops.cu", "ssd.cu", "ssd_chunk.cu", "attn_window.cu", "gemm_f32.cu"}
 
 COMPONENTS = {
-    "serve_hybrid": ["gemm_tcgen05.cu", "gemm2_tcgen05.cu", "elementwise.cu", "sampling.cu", "host_runtime.cu",
+    "serve_hybrid": ["gemm_tcgen05.cu", "gemm2_tcgen05.cu", "sampling.cu", "host_runtime.cu",
                      "hybrid_ops.cu", "ssd.cu", "ssd_chunk.cu", "attn_window.cu", "attn_window_tc.cu",
                      "attn_decode.cu", "gemm_f32.cu"],
 }

@@ -77,9 +77,9 @@ conv_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, const
 
 // The same for long batches: a thread slides down a run of tokens with the last TAPS - 1 inputs of its four channels in
 // registers, so every input is read once (and TAPS - 1 once more per run). A run may cross into another sequence.
-constexpr int CONV_RUN = 32, CONV_BATCH = 8;
+constexpr int CONV_RUN = 32, CONV_BATCH = 4;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 3)
 conv_run_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, const T* __restrict__ w,
                 const T* __restrict__ bias, T* __restrict__ out, const SsdDims d) {
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -95,13 +95,17 @@ conv_run_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, c
   int seq = -1;
   for (int t = t0; t < t1; t += CONV_BATCH) {
     float u[CONV_BATCH][4];
+    int ids[CONV_BATCH];
 #pragma unroll
     for (int j = 0; j < CONV_BATCH; ++j)
-      if (t + j < t1) load4(src.p + (size_t)(t + j) * src.ld + d.inner + c, u[j]);
+      if (t + j < t1) {
+        load4(src.p + (size_t)(t + j) * src.ld + d.inner + c, u[j]);
+        ids[j] = b.tok_seq[t + j];
+      }
 #pragma unroll
     for (int j = 0; j < CONV_BATCH; ++j) {
       if (t + j >= t1) break;
-      const int i = b.tok_seq[t + j];
+      const int i = ids[j];
       if (i != seq) {                                     // the run's first token, or another sequence begins
         seq = i;
         const int row0 = b.cu[i], o = t + j - row0;

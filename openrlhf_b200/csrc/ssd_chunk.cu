@@ -27,6 +27,13 @@ struct SsdChunkParams {
   __nv_bfloat16* y;           // [T, inner]
   Ragged b;
   int H, P, N, G, inner;
+  int pblocks;                // ceil(P / 64)
+  // long portions on few heads: segments of seg_chunks chunks run side by side (0: one CTA walks the whole portion).
+  // seg_state [n, H, n_seg, N, P] and seg_log2 [n, H, n_seg] hold every segment's own contribution to the state and its
+  // summed log2 decay after the first pass, the state at its start after the combination
+  int seg_chunks, n_seg;
+  float* seg_state;
+  float* seg_log2;
   int* status;
 };
 
@@ -61,6 +68,8 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
 // byte offset of 16-byte piece j of row r in a tile of 128-byte rows with the 128-byte swizzle
 __device__ __forceinline__ int sw128(int r, int j) { return r * 128 + ((j ^ (r & 7)) << 4); }
 
+// STATE_ONLY: the first pass over segments; only the recurrence runs (from zero), nothing is read out.
+template <bool STATE_ONLY>
 __global__ void __launch_bounds__(288, 2)
 ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p) {
   extern __shared__ __align__(1024) uint8_t smem[];
@@ -78,9 +87,17 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
   float* wsm = reinterpret_cast<float*>(smem + ScSmem::W_OFF);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int h = blockIdx.x, seq = blockIdx.y, p0 = blockIdx.z * SC_PB;
-  const int row0 = p.b.cu[seq], len = p.b.cu[seq + 1] - row0;
-  if (len <= 0) return;
+  const int h = blockIdx.x, seq = blockIdx.y, p0 = (blockIdx.z % p.pblocks) * SC_PB, seg = blockIdx.z / p.pblocks;
+  int row0 = p.b.cu[seq], len = p.b.cu[seq + 1] - row0;
+  bool last = true;                     // the CTA that ends the portion
+  if (p.seg_chunks > 0) {
+    const int off = seg * p.seg_chunks * SC_Q;
+    row0 += off;
+    len -= off;
+    last = len <= p.seg_chunks * SC_Q;
+    len = min(len, p.seg_chunks * SC_Q);
+  }
+  if (len <= 0 || (STATE_ONLY && last)) return;         // the last segment's contribution is nobody's start
   if (smem_u32(smem) & 1023) {          // the swizzled tiles need 1024-byte alignment; there is no room for slack
     if (threadIdx.x == 0 && p.status != nullptr) atomicCAS(p.status, 0, ERR_BAD_ARG);
     return;
@@ -129,7 +146,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
           tma_load_2d(smem + ScSmem::B_OFF + q * 16384, &tma, full, p.inner + g * p.N + q * 64, row0 + c * SC_Q);
       };
       load_b(0);
-      load_c(0);
+      if (!STATE_ONLY) load_c(0);
       const int kn = p.N >> 4;
       // descriptors of the first K step; a step adds its byte offset / 16 to the address field
       const uint64_t c_k = make_smem_desc_sw128(sc, 16, 1024), b_k = make_smem_desc_sw128(sb, 16, 1024);
@@ -137,34 +154,39 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
       const uint64_t s_mn = make_smem_desc_sw128(ss, 16384, 1024);
       for (int c = 0; c < n_chunks; ++c) {
         const uint32_t ph = c & 1;
-        if (!mbar_wait(full, ph, p.status, ERR_TIMEOUT_FULL) || !mbar_wait(c_full, ph, p.status, ERR_TIMEOUT_FULL)) break;
+        if (!mbar_wait(full, ph, p.status, ERR_TIMEOUT_FULL)) break;
+        if (!STATE_ONLY && !mbar_wait(c_full, ph, p.status, ERR_TIMEOUT_FULL)) break;
         tc_fence_after();
 #pragma unroll
         for (int k = 0; k < 8; ++k) {
           const uint64_t off = ((k >> 2) * 16384 + (k & 3) * 32) >> 4;
-          if (k < kn) umma_bf16(tm_g, c_k + off, b_k + off, id_g, k > 0);
+          if (!STATE_ONLY && k < kn) umma_bf16(tm_g, c_k + off, b_k + off, id_g, k > 0);
         }
         if (!mbar_wait(s_ready, ph, p.status, ERR_TIMEOUT_TMEM_EMPTY)) break;
         tc_fence_after();
         mbar_expect_tx(x_full, 16384);          // the previous chunk's y, staged in this tile, has been copied out
         tma_load_2d(smem + ScSmem::X_OFF, &tma, x_full, h * p.P + p0, row0 + c * SC_Q);
+        if (!STATE_ONLY) {
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const int k = i & 7;
-          const uint64_t off = ((k >> 2) * 16384 + (k & 3) * 32) >> 4;
-          if (k < kn) umma_bf16(tm_y, c_k + off, s_mn + (((i >> 3) * 16384 + k * 2048) >> 4), id_y, i > 0);
-        }
-        umma_commit(g_full);
-        if (c + 1 < n_chunks) {
-          if (!mbar_wait(g_full, ph, p.status, ERR_TIMEOUT_EMPTY)) break;
-          load_c(c + 1);
+          for (int i = 0; i < 16; ++i) {
+            const int k = i & 7;
+            const uint64_t off = ((k >> 2) * 16384 + (k & 3) * 32) >> 4;
+            if (k < kn) umma_bf16(tm_y, c_k + off, s_mn + (((i >> 3) * 16384 + k * 2048) >> 4), id_y, i > 0);
+          }
+          umma_commit(g_full);
+          if (c + 1 < n_chunks) {
+            if (!mbar_wait(g_full, ph, p.status, ERR_TIMEOUT_EMPTY)) break;
+            load_c(c + 1);
+          }
         }
         if (!mbar_wait(x_full, ph, p.status, ERR_TIMEOUT_FULL)) break;
-        if (!mbar_wait(m_ready, ph, p.status, ERR_TIMEOUT_TMEM_EMPTY)) break;
-        tc_fence_after();
+        if (!STATE_ONLY) {
+          if (!mbar_wait(m_ready, ph, p.status, ERR_TIMEOUT_TMEM_EMPTY)) break;
+          tc_fence_after();
 #pragma unroll
-        for (int i = 0; i < 16; ++i)
-          umma_bf16_ts(tm_y, tm_g + (i >> 3) * 64 + (i & 7) * 8, x_mn + (((i & 7) * 2048) >> 4), id_y, 1u);
+          for (int i = 0; i < 16; ++i)
+            umma_bf16_ts(tm_y, tm_g + (i >> 3) * 64 + (i & 7) * 8, x_mn + (((i & 7) * 2048) >> 4), id_y, 1u);
+        }
         if (!mbar_wait(xw_ready, ph, p.status, ERR_TIMEOUT_TMEM_EMPTY)) break;
         tc_fence_after();
 #pragma unroll
@@ -188,11 +210,16 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
     const int pn = min(SC_PB, p.P - p0);
     const float* dt = p.dt + (size_t)h * p.b.T + row0;
     float* gs = p.state + (((size_t)p.b.row[seq] * p.H + h) * p.N + t) * p.P + p0 + c0;
+    const size_t seg_i = p.seg_chunks > 0 ? ((size_t)seq * p.H + h) * p.n_seg + seg : 0;
+    float* ss = p.seg_state + (seg_i * p.N + t) * p.P + p0 + c0;
+    float log2_sum = 0.f;
     uint32_t r[32];
     {
-      const bool have = p.b.start[seq] != 0 && t < p.N;
+      const bool segs = p.seg_chunks > 0;
+      const bool have = !STATE_ONLY && t < p.N && (segs || p.b.start[seq] != 0);
+      const float* from = segs ? ss : gs;
 #pragma unroll
-      for (int j = 0; j < 32; ++j) r[j] = (have && c0 + j < pn) ? __float_as_uint(gs[j]) : 0u;
+      for (int j = 0; j < 32; ++j) r[j] = (have && c0 + j < pn) ? __float_as_uint(from[j]) : 0u;
       tmem_st_32x32b_x16(tm_s + lane_addr + c0, r);
       tmem_st_32x32b_x16(tm_s + lane_addr + c0 + 16, r + 16);
       tmem_st_wait();
@@ -224,6 +251,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
       const float gap2 = 0.f, gap1 = quarter > 2 ? b2 : 0.f, gap0 = quarter > 2 ? b1 + b2 : quarter > 1 ? b1 : 0.f;
       const float ahead = quarter == 0 ? b1 + b2 + b3 : quarter == 1 ? b2 + b3 : quarter == 2 ? b3 : 0.f;
       const float cum = pre + (quarter == 0 ? 0.f : b0 + gap0), total = b0 + b1 + b2 + b3;
+      log2_sum += total;
       // a block of 32 tokens in front of this row's weighs its token s with e^{sum behind s} dt_s, the same for all rows,
       // and the row adds the decay from the block's end to itself
       if (half == 0) wsm[t] = ex2(suf) * dtv;
@@ -235,15 +263,17 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
         const float decay = ex2(total);
         uint8_t* s_hi = smem + ScSmem::S_OFF;
         uint8_t* s_lo = s_hi + 16384;
+        if (!STATE_ONLY) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          uint32_t hi[4], lo[4];
+          for (int j = 0; j < 4; ++j) {
+            uint32_t hi[4], lo[4];
 #pragma unroll
-          for (int u = 0; u < 4; ++u)
-            split2(__uint_as_float(r[8 * j + 2 * u]), __uint_as_float(r[8 * j + 2 * u + 1]), hi[u], lo[u]);
-          const int off = sw128(t, half * 4 + j);
-          *reinterpret_cast<uint4*>(s_hi + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(s_lo + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+            for (int u = 0; u < 4; ++u)
+              split2(__uint_as_float(r[8 * j + 2 * u]), __uint_as_float(r[8 * j + 2 * u + 1]), hi[u], lo[u]);
+            const int off = sw128(t, half * 4 + j);
+            *reinterpret_cast<uint4*>(s_hi + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+            *reinterpret_cast<uint4*>(s_lo + off) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+          }
         }
 #pragma unroll
         for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * decay);
@@ -256,11 +286,13 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
         if (lane == 0) mbar_arrive(s_ready);
       }
       asm volatile("bar.sync 1, 256;" ::: "memory");        // wsm is complete
-      ok = ok && mbar_wait(g_full, ph, p.status, ERR_TIMEOUT_TMEM_FULL);
-      tc_fence_after();
+      if (!STATE_ONLY) {
+        ok = ok &&   mbar_wait(g_full, ph, p.status, ERR_TIMEOUT_TMEM_FULL);
+        tc_fence_after();
+      }
       // ---- weighted scores of the 32-column blocks half and half + 2 (blocks behind the diagonal are zero); all of G
       //      is read before M overwrites it
-      {
+      if (!STATE_ONLY) {
         uint32_t m_hi[2][16], m_lo[2][16];
 #pragma unroll
         for (int u = 0; u < 2; ++u) {
@@ -339,6 +371,7 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
       }
       ok = ok && mbar_wait(done, ph, p.status, ERR_TIMEOUT_TMEM_FULL);
       tc_fence_after();
+      if (STATE_ONLY) continue;
       // ---- y = Y + D x
       tmem_ld_32x32b_x32(tm_y + lane_addr + c0, r);
       tmem_ld_wait();
@@ -368,11 +401,13 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
     if (ok) {
       tmem_ld_32x32b_x32(tm_s + lane_addr + c0, r);         // all lanes take part
       tmem_ld_wait();
-      if (t < p.N && p.b.live(seq)) {
+      float* to = STATE_ONLY ? ss : gs;
+      if (t < p.N && (STATE_ONLY || (last && p.b.live(seq)))) {
 #pragma unroll
         for (int j = 0; j < 32; j += 4)
-          if (c0 + j < pn) *reinterpret_cast<uint4*>(gs + j) = make_uint4(r[j], r[j + 1], r[j + 2], r[j + 3]);
+          if (c0 + j < pn) *reinterpret_cast<uint4*>(to + j) = make_uint4(r[j], r[j + 1], r[j + 2], r[j + 3]);
       }
+      if (STATE_ONLY && threadIdx.x == 0 && p0 == 0) p.seg_log2[seg_i] = log2_sum;
     }
   }
 
@@ -390,6 +425,26 @@ ssd_chunk_kernel(const __grid_constant__ CUtensorMap tma, const SsdChunkParams p
   }
 }
 
+// Between the passes: every segment's contribution becomes the state at its start.
+__global__ void __launch_bounds__(256)
+ssd_segment_kernel(const SsdChunkParams p) {
+  const int h = blockIdx.x, seq = blockIdx.y, np = p.N * p.P;
+  const int len = p.b.cu[seq + 1] - p.b.cu[seq];
+  const int segs = (len + p.seg_chunks * SC_Q - 1) / (p.seg_chunks * SC_Q);
+  const size_t s0 = ((size_t)seq * p.H + h) * p.n_seg;
+  const float* gs = p.state + ((size_t)p.b.row[seq] * p.H + h) * np;
+  const bool fresh = p.b.start[seq] == 0;
+  for (int i = blockIdx.z * 256 + threadIdx.x; i < np; i += gridDim.z * 256) {
+    float v = fresh ? 0.f : gs[i];
+    for (int g = 0; g < segs; ++g) {
+      float* q = p.seg_state + (s0 + g) * np + i;
+      const float own = g + 1 < segs ? *q : 0.f;
+      *q = v;
+      if (g + 1 < segs) v = fmaf(ex2(p.seg_log2[s0 + g]), v, own);
+    }
+  }
+}
+
 }  // namespace b200
 
 using namespace b200;
@@ -400,22 +455,37 @@ extern "C" int b200_ssd_chunk_fits(int H, int P, int N, int G) {
   return cc % 8 == 0 && P % 8 == 0 && inner % 8 == 0 && N % 16 == 0 && N <= 128 ? 1 : 0;
 }
 
-// bf16 scan of a ragged batch; same contract as b200_ssd_scan with f32 = 0.
+// bf16 scan of a ragged batch; same contract as b200_ssd_scan with f32 = 0. seg_chunks > 0: portions are cut into n_seg
+// segments of that many chunks (n_seg * seg_chunks * 128 tokens cover the longest); seg_state holds n * H * n_seg * N * P
+// floats, seg_log2 n * H * n_seg.
 extern "C" int b200_ssd_chunk(const void* xbc, const float* dt, const int* cu, const int* start, const int* row,
                               const int* active, const int* tok_seq, int n, int T, const void* a_log, const void* dskip,
-                              float* state, void* y, int H, int P, int N, int G, int* status, void* stream) {
+                              float* state, void* y, int H, int P, int N, int G, int seg_chunks, int n_seg,
+                              float* seg_state, float* seg_log2, int* status, void* stream) {
   if (T <= 0 || n <= 0) return 0;
+  if (seg_chunks > 0 && (n_seg < 1 || seg_state == nullptr || seg_log2 == nullptr ||
+                         (reinterpret_cast<uintptr_t>(seg_state) & 15))) return -11;
   if (H % G || n > 65535 || !b200_ssd_chunk_fits(H, P, N, G)) return -10;
   if ((reinterpret_cast<uintptr_t>(xbc) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(state)) & 15) return -12;
   const int inner = H * P, cc = inner + 2 * G * N;
   CUtensorMap tm;
   if (int r = make_tmap_bf16_2d(&tm, xbc, T, cc, cc, SC_Q, 64)) return r;
-  static std::atomic<unsigned long long> configured{0};
-  if (!set_max_smem_once(configured, ssd_chunk_kernel, ScSmem::TOTAL)) return -2;
+  static std::atomic<unsigned long long> c0{0}, c1{0};
+  if (!set_max_smem_once(c0, ssd_chunk_kernel<false>, ScSmem::TOTAL)) return -2;
+  if (!set_max_smem_once(c1, ssd_chunk_kernel<true>, ScSmem::TOTAL)) return -2;
   SsdChunkParams p;
   p.dt = dt; p.a_log = reinterpret_cast<const __nv_bfloat16*>(a_log); p.dskip = reinterpret_cast<const __nv_bfloat16*>(dskip);
   p.state = state; p.y = reinterpret_cast<__nv_bfloat16*>(y); p.b = make_ragged(cu, start, row, active, tok_seq, n, T);
   p.H = H; p.P = P; p.N = N; p.G = G; p.inner = inner; p.status = status;
-  ssd_chunk_kernel<<<dim3(H, n, (P + SC_PB - 1) / SC_PB), 288, ScSmem::TOTAL, reinterpret_cast<cudaStream_t>(stream)>>>(tm, p);
+  p.pblocks = (P + SC_PB - 1) / SC_PB;
+  p.seg_chunks = seg_chunks > 0 ? seg_chunks : 0; p.n_seg = seg_chunks > 0 ? n_seg : 1;
+  p.seg_state = seg_state; p.seg_log2 = seg_log2;
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  const dim3 grid(H, n, p.pblocks * p.n_seg);
+  if (p.seg_chunks > 0) {
+    ssd_chunk_kernel<true><<<grid, 288, ScSmem::TOTAL, st>>>(tm, p);
+    ssd_segment_kernel<<<dim3(H, n, (N * P + 255) / 256), 256, 0, st>>>(p);
+  }
+  ssd_chunk_kernel<false><<<grid, 288, ScSmem::TOTAL, st>>>(tm, p);
   return cudaGetLastError() == cudaSuccess ? 0 : -3;
 }

@@ -178,9 +178,10 @@ CHUNK_MIN = 8      # portions of at least this many tokens take the tensor-core 
 
 
 def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, m, a_log: torch.Tensor, d: torch.Tensor, state: torch.Tensor,
-             y: torch.Tensor, batch: StepBatch, chunked: bool | None = None) -> None:
+             y: torch.Tensor, batch: StepBatch, chunked: bool | None = None, segments: int | None = None) -> None:
     """Recurrence over the convolved inputs xbc [T, channels] and step sizes dt fp32 [heads, T]; y [T, inner]. `chunked`
-    picks the tensor-core kernel (bf16, sizes it covers) or the token-by-token one; None: by portion length."""
+    picks the tensor-core kernel (bf16, sizes it covers) or the token-by-token one; None: by portion length. `segments`:
+    how many pieces of a portion the tensor-core kernel runs side by side; None: as many as fill the GPU."""
     L = _lib.lib()
     seqs = (_p(batch.cu), _p(batch.start), _p(batch.row), _p(batch.active), _p(batch.tok_seq), _i(batch.n), _i(batch.T))
     H, P, N, G = _i(m.heads), _i(m.vdim), _i(m.state), _i(m.groups)
@@ -189,7 +190,19 @@ def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, m, a_log: torch.Tensor, d: tor
         chunked = fits and batch.max_new >= CHUNK_MIN
     if chunked:
         assert fits, "sizes outside the tensor-core scan"
-        _lib.check_rc(L.b200_ssd_chunk(_p(xbc), _p(dt), *seqs, _p(a_log), _p(d), _p(state), _p(y), H, P, N, G,
+        chunks = (batch.max_new + 127) // 128
+        if segments is None:
+            # a segment costs a second, cheaper pass over its tokens: only when heads and sequences leave SMs idle
+            ctas = m.heads * batch.n * ((m.vdim + 63) // 64)
+            segments = min(2 * 148 // ctas, chunks // 4) if ctas <= 100 else 1
+        per = (chunks + segments - 1) // segments if segments > 1 else 0
+        nseg = (chunks + per - 1) // per if per else 1
+        seg_state = seg_log2 = None
+        if per:
+            seg_state = torch.empty(batch.n, m.heads, nseg, m.state, m.vdim, dtype=torch.float32, device=xbc.device)
+            seg_log2 = torch.empty(batch.n, m.heads, nseg, dtype=torch.float32, device=xbc.device)
+        _lib.check_rc(L.b200_ssd_chunk(_p(xbc), _p(dt), *seqs, _p(a_log), _p(d), _p(state), _p(y), H, P, N, G, _i(per),
+                                       _i(nseg), _p(seg_state), _p(seg_log2),
                                        _p(_lib.status_word(xbc.device)), _lib.stream_ptr()), "ssd_chunk")
     else:
         _lib.check_rc(L.b200_ssd_scan(_p(xbc), _p(dt), *seqs, _p(a_log), _p(d), _p(state), _p(y), H, P, N, G, _i(m.conv),

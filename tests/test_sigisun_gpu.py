@@ -198,13 +198,19 @@ def test_tensor_core_scan_keeps_32_bit_state():
         a_log = torch.linspace(-4, 3, spec.heads, device=DEV).bfloat16()
         d = torch.randn(spec.heads, device=DEV, generator=g).bfloat16()
         s0 = torch.randn(len(lens) + 1, spec.heads, spec.state, spec.vdim, device=DEV, generator=g)
-        s32, s16 = s0.clone(), s0.clone()
+        s32, s16, s_seg = s0.clone(), s0.clone(), s0.clone()
         y32 = torch.empty(T, spec.inner, device=DEV)
         y16 = torch.empty(T, spec.inner, device=DEV, dtype=torch.bfloat16)
         H.ssd_scan(xbc.float(), dt, spec, a_log.float(), d.float(), s32, y32, batch, chunked=False)
         H.ssd_scan(xbc, dt, spec, a_log, d, s16, y16, batch, chunked=True)
         close(s16, s32.double().cpu(), torch.float32, tol32=2.0 ** -17)      # two bf16 pieces of every 32-bit operand
         close(y16, y32.double().cpu(), torch.bfloat16, tol16=4e-3)
+        for segments in (2, 3):                    # pieces of a portion side by side
+            s_seg.copy_(s0)
+            y16.zero_()
+            H.ssd_scan(xbc, dt, spec, a_log, d, s_seg, y16, batch, chunked=True, segments=segments)
+            close(s_seg, s32.double().cpu(), torch.float32, tol32=2.0 ** -16)
+            close(y16, y32.double().cpu(), torch.bfloat16, tol16=4e-3)
 
 
 ATTN = [attn(6, 2, 64, 64, 0.2, 96 + 5, 3, 32), attn(3, 1, 22, 13, 0.3, 5, 1, 6), attn(4, 4, 128, 96, 0.1, 128, 0),
