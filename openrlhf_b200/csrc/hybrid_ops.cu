@@ -120,9 +120,10 @@ __global__ void softcap_kernel(float* __restrict__ x, long long n4, float cap, f
 // layer's cache. Channels [0, rot) of a head rotate in pairs (i, i + rot/2) with the (cos, sin) row of the token's
 // position; the rest pass. q -> q_out [T, H, dk_ld]; k, v -> cache slot. Cache and q rows are padded to dk_ld / dv_ld
 // (their padding stays zero). One thread per element pair; ff columns are squared-ReLU'd into `ff_dst`.
-// The same, four channels at a time (rot / 2, dk - rot and dv multiples of 4).
-template <typename T>
-__global__ void __launch_bounds__(HY_THREADS)
+// The same, four channels at a time (rot / 2, dk - rot and dv multiples of 4) for NT consecutive tokens per thread; all
+// loads of a thread are issued before its first store.
+template <typename T, int NT>
+__global__ void __launch_bounds__(HY_THREADS, 4)
 rope_write4_kernel(const Proj<T> src, const int* __restrict__ pos, const int* __restrict__ slots,
                    const float2* __restrict__ table, int max_pos, T* __restrict__ q_out, T* __restrict__ k_cache,
                    T* __restrict__ v_cache, int n_tok, int H, int G, int dk, int dv, int dk_ld, int dv_ld, int rot,
@@ -132,48 +133,69 @@ rope_write4_kernel(const Proj<T> src, const int* __restrict__ pos, const int* __
   const int half = rot >> 1;
   const int per_qk = (half + (dk - rot)) >> 2;
   const int n_qk = (H + G) * per_qk, n_v = (G * dv) >> 2, n_f = ff >> 2;
-  const int per_tok = n_qk + n_v + n_f;
-  const int step = gridDim.x * HY_THREADS;
-  const long long total = (long long)n_tok * per_tok;
-  for (long long idx = blockIdx.x * (long long)HY_THREADS + threadIdx.x; idx < total; idx += step) {
-    const int t = (int)(idx / per_tok);
-    int e = (int)(idx - (long long)t * per_tok);
-    float u[4];
-    if (e < n_qk) {
-      const int head = e / per_qk, i = (e - head * per_qk) * 4;
-      T* dst = head < H ? q_out + ((size_t)t * H + head) * dk_ld : k_cache + ((size_t)slots[t] * G + (head - H)) * dk_ld;
-      const int c0 = head * dk;
-      if (i < half) {
-        float v[4], a[4], b[4], cs[8];
-        src.get4(t, c0 + i, u);
-        src.get4(t, c0 + i + half, v);
+  int e = blockIdx.y * HY_THREADS + threadIdx.x;
+  if (e >= n_qk + n_v + n_f) return;
+  const int t0 = blockIdx.x * NT;
+  float u[NT][4];
+  if (e < n_qk) {
+    const int head = e / per_qk, i = (e - head * per_qk) * 4, c0 = head * dk;
+    const bool turns = i < half;
+    float v[NT][4], cs[NT][8];
+    int slot[NT];
+#pragma unroll
+    for (int k = 0; k < NT; ++k) {
+      const int t = min(t0 + k, n_tok - 1);
+      src.get4(t, c0 + i + (turns ? 0 : half), u[k]);
+      if (head >= H) slot[k] = slots[t];
+      if (turns) {
+        src.get4(t, c0 + i + half, v[k]);
         int p = pos[t];
         p = p < 0 ? 0 : (p >= max_pos ? max_pos - 1 : p);
         const float* row = reinterpret_cast<const float*>(table + (size_t)p * half + i);
-        load4(row, cs);
-        load4(row + 4, cs + 4);
+        load4(row, cs[k]);
+        load4(row + 4, cs[k] + 4);
+      }
+    }
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          a[k] = u[k] * cs[2 * k] - v[k] * cs[2 * k + 1];
-          b[k] = v[k] * cs[2 * k] + u[k] * cs[2 * k + 1];
+    for (int k = 0; k < NT; ++k) {
+      if (t0 + k >= n_tok) break;
+      T* dst = head < H ? q_out + ((size_t)(t0 + k) * H + head) * dk_ld : k_cache + ((size_t)slot[k] * G + (head - H)) * dk_ld;
+      if (turns) {
+        float a[4], b[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          a[j] = u[k][j] * cs[k][2 * j] - v[k][j] * cs[k][2 * j + 1];
+          b[j] = v[k][j] * cs[k][2 * j] + u[k][j] * cs[k][2 * j + 1];
         }
         store4(dst + i, a);
         store4(dst + i + half, b);
       } else {
-        src.get4(t, c0 + i + half, u);
-        store4(dst + i + half, u);
+        store4(dst + i + half, u[k]);
       }
-    } else if (e < n_qk + n_v) {
-      e = (e - n_qk) * 4;
-      const int g = e / dv;
-      src.get4(t, (H + G) * dk + e, u);
-      store4(v_cache + ((size_t)slots[t] * G + g) * dv_ld + (e - g * dv), u);
-    } else {
-      e = (e - n_qk - n_v) * 4;
-      src.get4(t, ff_col + e, u);
+    }
+  } else if (e < n_qk + n_v) {
+    e = (e - n_qk) * 4;
+    const int g = e / dv;
+    int slot[NT];
 #pragma unroll
-      for (int k = 0; k < 4; ++k) { const float r = fmaxf(u[k], 0.f); u[k] = r * r; }
-      store4(ff_dst + (size_t)t * ff_ld + e, u);
+    for (int k = 0; k < NT; ++k) {
+      const int t = min(t0 + k, n_tok - 1);
+      src.get4(t, (H + G) * dk + e, u[k]);
+      slot[k] = slots[t];
+    }
+#pragma unroll
+    for (int k = 0; k < NT; ++k)
+      if (t0 + k < n_tok) store4(v_cache + ((size_t)slot[k] * G + g) * dv_ld + (e - g * dv), u[k]);
+  } else {
+    e = (e - n_qk - n_v) * 4;
+#pragma unroll
+    for (int k = 0; k < NT; ++k) src.get4(min(t0 + k, n_tok - 1), ff_col + e, u[k]);
+#pragma unroll
+    for (int k = 0; k < NT; ++k) {
+      if (t0 + k >= n_tok) break;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) { const float r = fmaxf(u[k][j], 0.f); u[k][j] = r * r; }
+      store4(ff_dst + (size_t)(t0 + k) * ff_ld + e, u[k]);
     }
   }
 }
@@ -345,14 +367,19 @@ extern "C" int b200_rope_write(const void* p, const float* ws, int splits, long 
   if (rot % 2 || rot > dk || dk_ld < dk || dv_ld < dv || ff % 4 || ff_col % 4 || ld % 4 || ff_ld % 4 || slab % 4) return -10;
   const long long work = (long long)n_tok * ((H + G) * (rot / 2 + dk - rot) + G * dv + ff / 4);
   const bool vec = rot % 8 == 0 && (dk - rot) % 4 == 0 && dv % 4 == 0;
-  const int grid = hy_grid(vec ? work / 4 : work, 148 * 16);
+  const int grid = hy_grid(work, 148 * 16);
+  const int nt = n_tok >= 512 ? 2 : 1;
+  const dim3 grid4((n_tok + nt - 1) / nt, (unsigned)(work / n_tok / (4 * HY_THREADS) + 1));
   cudaError_t e;
 #define ROPE_ARGS(TT)                                                                                                 \
   make_proj<TT>(p, ws, splits, slab, ld), pos, slots, (const float2*)table, max_pos, (TT*)q_out, (TT*)k_cache,        \
       (TT*)v_cache, n_tok, H, G, dk, dv, dk_ld, dv_ld, rot, ff_col, ff, (TT*)ff_dst, ff_ld
   if (vec) {
-    if (f32) e = launch_pdl(rope_write4_kernel<float>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(float));
-    else e = launch_pdl(rope_write4_kernel<__nv_bfloat16>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(__nv_bfloat16));
+#define ROPE4(TT, NT) \
+  launch_pdl(rope_write4_kernel<TT, NT>, grid4, dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(TT))
+    if (f32) e = nt == 2 ? ROPE4(float, 2) : ROPE4(float, 1);
+    else e = nt == 2 ? ROPE4(__nv_bfloat16, 2) : ROPE4(__nv_bfloat16, 1);
+#undef ROPE4
   } else if (f32) e = launch_pdl(rope_write_kernel<float>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(float));
   else e = launch_pdl(rope_write_kernel<__nv_bfloat16>, dim3(grid), dim3(HY_THREADS), (size_t)0, HY_STREAM(stream), ROPE_ARGS(__nv_bfloat16));
 #undef ROPE_ARGS

@@ -79,7 +79,7 @@ conv_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, const
 // registers, so every input is read once (and TAPS - 1 once more per run). A run may cross into another sequence.
 constexpr int CONV_RUN = 32, CONV_BATCH = 4;
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(256, 3)
+__global__ void __launch_bounds__(128, 6)
 conv_run_kernel(const Proj<T> src, const Ragged b, const T* __restrict__ ring, const T* __restrict__ w,
                 const T* __restrict__ bias, T* __restrict__ out, const SsdDims d) {
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
@@ -296,12 +296,12 @@ static int launch_conv(const Proj<T>& src, const Ragged& b, T* ring, const T* w,
                        float* dt, const SsdDims& d, cudaStream_t st) {
   const bool vec = d.cc % 4 == 0 && d.inner % 4 == 0 && src.ld % 4 == 0 && src.slab % 4 == 0;
   if (vec && src.ws == nullptr && b.T >= 64 && d.taps >= 1 && d.taps <= 4) {
-    const dim3 grid((d.cc / 4 + 255) / 256, (b.T + CONV_RUN - 1) / CONV_RUN);
+    const dim3 grid((d.cc / 4 + 127) / 128, (b.T + CONV_RUN - 1) / CONV_RUN);
     if (grid.y > 65535) return -10;
-    if (d.taps == 1) conv_run_kernel<T, 1><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
-    else if (d.taps == 2) conv_run_kernel<T, 2><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
-    else if (d.taps == 3) conv_run_kernel<T, 3><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
-    else conv_run_kernel<T, 4><<<grid, 256, 0, st>>>(src, b, ring, w, bias, out, d);
+    if (d.taps == 1) conv_run_kernel<T, 1><<<grid, 128, 0, st>>>(src, b, ring, w, bias, out, d);
+    else if (d.taps == 2) conv_run_kernel<T, 2><<<grid, 128, 0, st>>>(src, b, ring, w, bias, out, d);
+    else if (d.taps == 3) conv_run_kernel<T, 3><<<grid, 128, 0, st>>>(src, b, ring, w, bias, out, d);
+    else conv_run_kernel<T, 4><<<grid, 128, 0, st>>>(src, b, ring, w, bias, out, d);
     dt_kernel<T><<<(b.T + 31) / 32, 256, 0, st>>>(src, dt_bias, dt, b.T, d);
     if (cudaGetLastError() != cudaSuccess) return -3;
     if (d.taps > 1) conv_ring_kernel<T><<<dim3((d.cc + 255) / 256, b.n), 256, 0, st>>>(src, b, ring, d);

@@ -111,3 +111,26 @@ def test_fixed_length_rows_decode_in_long_bursts_with_identical_outputs(model, p
     # 90 tokens: rows that may stop on EOS start with bursts of 4 steps and grow to 8 and 16 while nobody finishes
     # (4 + 4 + 8 + 8 + 16 ...: about nine calls); rows that cannot stop early run 32 steps at a time from the start
     assert 7 <= calls["eos"] <= 12 and calls["fixed"] <= 6 and calls["fixed"] < calls["eos"], calls
+
+
+def test_given_tokens_in_portions_give_the_models_logits(model, prompts):
+    """``extend``: sequences fed in portions of any size, side by side, against one forward pass of each."""
+    eng = RolloutEngine(model, max_num_seqs=3, max_model_len=512, num_pages=9)
+    seqs = {"a": prompts[1], "b": prompts[3], "c": prompts[0]}
+    want = {}
+    for k, t in seqs.items():
+        n = len(t)
+        h, _ = model(torch.tensor(t), torch.arange(n, dtype=torch.int32), torch.tensor([0, n], dtype=torch.int32), n)
+        want[k] = model.logits(h).detach()
+    at = dict.fromkeys(seqs, 0)
+    for a, b, c in ((130, 1, 2), (1, 64, 1), (2, 1, 0), (100, 70, 1), (67, 4, 1)):
+        entries = [(k, seqs[k][at[k]:at[k] + n], list(range(n))) for k, n in zip("abc", (a, b, c)) if n]
+        lg, o = eng.extend(entries), 0
+        for k, part, _ in entries:
+            assert (lg[o:o + len(part)] - want[k][at[k]:at[k] + len(part)]).abs().max() < 1e-3, (k, at[k])
+            o += len(part)
+            at[k] += len(part)
+    assert at == {k: len(t) for k, t in seqs.items()}
+    for k in seqs:
+        eng.finish(k)
+    assert eng.blocks.num_free() == 9 - 1 and not eng.has_unfinished()

@@ -98,6 +98,20 @@ def test_softcap_embedding_and_fp32_product():
     assert torch.equal(H.embed(ids, tab.to(DEV)).cpu(), tab[ids.cpu()].float())
 
 
+@pytest.mark.parametrize("M,N,K,col0", [(300, 352, 72, 224), (2048, 4352, 512, 2304), (1500, 8224, 264, 32)])
+def test_input_projection_with_squared_relu_epilogue(M, N, K, col0):
+    """The single-CTA and the CTA-pair GEMM: columns before col0 as they are, the rest as relu^2 into wider rows."""
+    from openrlhf_b200.ops.gemm import gemm_relu2
+
+    x, w = rnd(M, K, seed=1), rnd(N, K, seed=2)
+    act = torch.full((M, N - col0 + 64), 5.0, dtype=torch.bfloat16, device=DEV)
+    got = gemm_relu2(x.to(DEV), w.to(DEV), col0, act[:, 32:32 + N - col0])
+    want = x.double() @ w.double().T
+    close(got, want[:, :col0], torch.bfloat16)
+    close(act[:, 32:32 + N - col0], torch.relu(want[:, col0:]) ** 2, torch.bfloat16)
+    assert (act[:, :32] == 5).all() and (act[:, 32 + N - col0:] == 5).all()
+
+
 MAMBAS = [mamba(4, 64, 128, 2, 4, 2), mamba(5, 7, 11, 5, 1, 5), mamba(3, 48, 16, 1, 3, 1), mamba(2, 128, 64, 1, 2, 4),
           mamba(6, 24, 96, 3, 5, 3), mamba(2, 40, 144, 2, 4, 1)]
 
