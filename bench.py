@@ -83,7 +83,7 @@ def parse():
                     help="auto: after the default config, measure the other configs in child processes if time allows")
     ap.add_argument("--serving", default=None, metavar="SIZES",
                     help="instead: prefill and decode throughput of the hybrid design beside the dense transformer of equal "
-                         "size, e.g. 1b or 1b,8b (bench/serving.py); one GPU")
+                         "size, e.g. 1b or 1b,3b,8b (bench/serving.py); one GPU")
     return ap.parse_args()
 
 

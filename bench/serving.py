@@ -10,7 +10,7 @@ import statistics
 
 import torch
 
-SIZES = {"1b": "sigisun-1b", "8b": "sigisun-8b"}
+SIZES = {"1b": "sigisun-1b", "3b": "sigisun-3b", "8b": "sigisun-8b"}
 
 
 def dense_twin(cfg):

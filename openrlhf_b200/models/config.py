@@ -222,5 +222,6 @@ PRESETS: dict[str, ModelConfig] = {
 PRESETS.update({
     "tiny-sigisun": sigisun_preset(192, 6, 6, 32, 48, 2, 6, 2, 48, 40, 3, 224, 512),
     "sigisun-1b": sigisun_preset(2048, 24, 64, 64, 128, 1, 16, 4, 128, 1024, 4, 4096, 65536),
+    "sigisun-3b": sigisun_preset(3072, 30, 96, 64, 128, 2, 24, 8, 128, 1024, 4, 8192, 128256),
     "sigisun-8b": sigisun_preset(4096, 36, 128, 64, 128, 8, 32, 8, 128, 2048, 4, 11008, 128256),
 })
