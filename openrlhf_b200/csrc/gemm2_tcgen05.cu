@@ -516,7 +516,7 @@ extern "C" int b200_gemm2_bf16(const void* A, const void* B, void* C, const void
                          bn, 0, nullptr, 0, status, stream_);
 }
 
-// Split output with relu^2 on the columns from act_col0 on; same contract as b200_gemm_bf16_relu2.
+// Split output with relu^2 on the columns from act_col0 on; same arguments as b200_gemm_bf16_relu2.
 extern "C" int b200_gemm2_bf16_relu2(const void* A, const void* B, void* C, void* C2, int M, int N, int K, int lda, int ldb,
                                      int ldc, int ldc2, int act_col0, int bn, int* status, void* stream_) {
   if (act_col0 <= 0 || act_col0 % 32 || N % 32 || ldc2 % 8 || (reinterpret_cast<uintptr_t>(C2) & 15)) return -10;

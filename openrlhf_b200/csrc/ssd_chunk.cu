@@ -455,7 +455,7 @@ extern "C" int b200_ssd_chunk_fits(int H, int P, int N, int G) {
   return cc % 8 == 0 && P % 8 == 0 && inner % 8 == 0 && N % 16 == 0 && N <= 128 ? 1 : 0;
 }
 
-// bf16 scan of a ragged batch; same contract as b200_ssd_scan with f32 = 0. seg_chunks > 0: portions are cut into n_seg
+// bf16 scan of a ragged batch; like b200_ssd_scan with f32 = 0. seg_chunks > 0: portions are cut into n_seg
 // segments of that many chunks (n_seg * seg_chunks * 128 tokens cover the longest); seg_state holds n * H * n_seg * N * P
 // floats, seg_log2 n * H * n_seg.
 extern "C" int b200_ssd_chunk(const void* xbc, const float* dt, const int* cu, const int* start, const int* row,
